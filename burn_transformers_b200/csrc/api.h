@@ -175,6 +175,10 @@ int bt_selective_scan(const void* x, long long x_row_stride, const void* z, long
                       const float* d_skip, float* state, const int* slots, const int* seq_start, void* out,
                       long long out_row_stride, int n_seqs, int channels, int n_state, float out_scale, int piece,
                       int max_pieces, float* ends, int dtype, cudaStream_t stream);
+// The gated average of a minimal GRU (csrc/min_gru.cu).
+int bt_min_gru(const void* proj, long long row_stride, int z_off, int x_off, int g_off, const float* z_bias,
+               const float* x_bias, float* state, const int* slots, const int* seq_start, void* out,
+               long long out_row_stride, int n_seqs, int width, int max_new, int dtype, cudaStream_t stream);
 int bt_rotary_interleaved(const void* src, long long src_row_stride, int src_vec_stride, void* dst,
                           long long dst_row_stride, int dst_vec_stride, const int* positions, const float* inv_freq,
                           int n_tokens, int n_vecs, int len, int dims, int dtype, cudaStream_t stream);
@@ -196,8 +200,8 @@ int bt_mlstm_chunked(const void* proj, long long row_stride, int q_off, int k_of
                      long long n_rows, int max_new, int n_seqs, int n_heads, int dim, int vdim, int dtype,
                      cudaStream_t stream);
 int bt_moe_route(const void* x, long long x_row_stride, const void* router, int n_tokens, int K, int E, int top,
-                 int n_groups, int keep, float scale, int softmax, const float* choice_bias, int normalise, int* ids,
-                 float* weights, int dtype, cudaStream_t stream);
+                 int n_groups, int keep, float scale, int rule, const float* logit_bias, const float* choice_bias, int normalise,
+                 int* ids, float* weights, int dtype, cudaStream_t stream);
 int bt_moe_tile_rows();
 int bt_moe_sort(const int* ids, int total, int E, int* offsets, int* tile_first, int* order, int* place,
                 cudaStream_t stream);

@@ -136,8 +136,8 @@ __device__ __forceinline__ float gelu_erf(float x) {
   return 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
 }
 
-// kActSwishClamp is a rule for a (gate, up) pair, see gated_pair; alone it leaves a value as it is.
-enum Activation : int { kActNone = 0, kActGeluTanh = 1, kActGeluErf = 2, kActSwishClamp = 3 };
+// kActSwishClamp and kActSwish are rules for a (gate, up) pair, see gated_pair; alone they leave a value as it is.
+enum Activation : int { kActNone = 0, kActGeluTanh = 1, kActGeluErf = 2, kActSwishClamp = 3, kActSwish = 4 };
 
 __device__ __forceinline__ float apply_activation(float v, int act) {
   if (act == kActGeluTanh) return gelu_tanh(v);
@@ -145,14 +145,15 @@ __device__ __forceinline__ float apply_activation(float v, int act) {
   return v;
 }
 
-// The hidden value of a gated feed-forward from its pair (gate g, up u): act(g) * u, or, for kActSwishClamp,
-// g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit) and u' = u clamped to [-limit, limit].
+// The hidden value of a gated feed-forward from its pair (gate g, up u): act(g) * u; for kActSwish g sigmoid(g) * u; for
+// kActSwishClamp g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit) and u' = u clamped to [-limit, limit].
 __device__ __forceinline__ float gated_pair(float g, float u, int act, float limit) {
   if (act == kActSwishClamp) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
   }
+  if (act == kActSwish) return g / (1.f + expf(-g)) * u;
   return apply_activation(g, act) * u;
 }
 

@@ -4,8 +4,10 @@
 //   moe_route    per token: z = W_r x in 32-bit, s = sigmoid(z); experts lie in `n_groups` equal groups of neighbours, a
 //                group's score is the sum of its two largest s, only the `keep` best groups may give experts; the `top`
 //                largest s among those are chosen (equal scores: the lower index); weights s / (sum of the chosen + 1e-20)
-//                * scale.  With `softmax` the scores are softmax(z) over all experts instead; `choice_bias` [E] is added
-//                to the scores for the choice only; without `normalise` the weights are the chosen scores as they are.
+//                * scale.  `logit_bias` [E] is added to z.  With rule 1 the scores are softmax(z) over all experts
+//                instead; with rule 2 they are z itself and the weights softmax over the chosen z, times scale;
+//                `choice_bias` [E] is added to the scores for the choice only; without `normalise` the weights are the
+//                chosen scores as they are (rules 0 and 1).
 //   moe_sort     counts the pairs per expert, gives each pair a row in expert order, and numbers the row tiles
 //                (tiles never straddle two experts).
 //   moe_expert_in   hidden[r] = pair rule(gate_e x, up_e x) for the rows of expert e (x gathered by the pair's token), or,
@@ -32,6 +34,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 }
 
 constexpr int ROUTE_WARPS = 4;
+constexpr int kRouteSigmoid = 0, kRouteSoftmax = 1, kRouteChosen = 2;
 
 // A 16-byte piece of a row as 32-bit numbers.
 __device__ __forceinline__ void load_piece(const float* p, float (&o)[4]) {
@@ -67,8 +70,8 @@ __device__ __forceinline__ void unpack_piece(const uint4& v, float (&o)[8]) {
 template <typename T, int NP>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const T* __restrict__ x, long long x_row_stride, const T* __restrict__ router, int n_tokens, int K, int E,
-                 int top, int n_groups, int keep, float scale, int softmax, const float* __restrict__ choice_bias,
-                 int normalise, int* __restrict__ ids, float* __restrict__ weights) {
+                 int top, int n_groups, int keep, float scale, int rule, const float* __restrict__ logit_bias,
+                 const float* __restrict__ choice_bias, int normalise, int* __restrict__ ids, float* __restrict__ weights) {
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float* score = sm + (size_t)warp * 3 * E;   // [E] sigmoid scores
@@ -110,7 +113,10 @@ moe_route_kernel(const T* __restrict__ x, long long x_row_stride, const T* __res
           for (int u = 0; u < V; ++u) acc = fmaf(xv[i][u], wv[u], acc);
         }
         acc = warp_sum(acc);
-        if (lane == 0 && e0 + j < E) score[e0 + j] = softmax ? acc : 1.f / (1.f + expf(-acc));
+        if (lane == 0 && e0 + j < E) {
+          if (logit_bias != nullptr) acc += logit_bias[e0 + j];
+          score[e0 + j] = rule != kRouteSigmoid ? acc : 1.f / (1.f + expf(-acc));
+        }
       }
     }
   } else {
@@ -124,13 +130,16 @@ moe_route_kernel(const T* __restrict__ x, long long x_row_stride, const T* __res
       }
 #pragma unroll
       for (int j = 0; j < EB; ++j) {
-        const float z = warp_sum(acc[j]);
-        if (lane == 0 && e0 + j < E) score[e0 + j] = softmax ? z : 1.f / (1.f + expf(-z));
+        float z = warp_sum(acc[j]);
+        if (lane == 0 && e0 + j < E) {
+          if (logit_bias != nullptr) z += logit_bias[e0 + j];
+          score[e0 + j] = rule != kRouteSigmoid ? z : 1.f / (1.f + expf(-z));
+        }
       }
     }
   }
   __syncwarp();
-  if (softmax) {
+  if (rule == kRouteSoftmax) {
     float top_z = -INFINITY;
     for (int e = lane; e < E; e += 32) top_z = fmaxf(top_z, score[e]);
     top_z = warp_max(top_z);
@@ -183,6 +192,14 @@ moe_route_kernel(const T* __restrict__ x, long long x_row_stride, const T* __res
     }
     sum += v;
     __syncwarp();
+  }
+  if (rule == kRouteChosen) {        // (up to 32 choices, a lane each; without a choice_bias the first one is the largest)
+    const long long at = (long long)t * top + lane;
+    const float z = lane < top ? weights[at] : -INFINITY;
+    const float grown = expf(z - warp_max(z));
+    const float denom = warp_sum(grown);
+    if (lane < top) weights[at] = grown / denom * scale;
+    return;
   }
   if (normalise && lane < top) {
     const long long at = (long long)t * top + lane;
@@ -552,12 +569,14 @@ moe_combine_kernel(const float* __restrict__ part, const int* __restrict__ place
 }  // namespace bt
 
 extern "C" int bt_moe_route(const void* x, long long x_row_stride, const void* router, int n_tokens, int K, int E, int top,
-                            int n_groups, int keep, float scale, int softmax, const float* choice_bias, int normalise,
-                            int* ids, float* weights, int dtype, cudaStream_t stream) {
+                            int n_groups, int keep, float scale, int rule, const float* logit_bias,
+                            const float* choice_bias, int normalise, int* ids, float* weights, int dtype, cudaStream_t stream) {
   using namespace bt;
   BT_CHECK(n_tokens >= 0 && K > 0 && E > 0 && E <= 1024 && top > 0 && top <= 32 && n_groups > 0 && E % n_groups == 0 &&
                keep > 0 && keep <= n_groups && top <= keep * (E / n_groups),
            "moe_route: bad sizes experts=%d (up to 1024) top=%d (up to 32) groups=%d keep=%d", E, top, n_groups, keep);
+  BT_CHECK(rule >= kRouteSigmoid && rule <= kRouteChosen && (rule != kRouteChosen || (n_groups == 1 && normalise)),
+           "moe_route: rule %d; a softmax over the chosen goes with one group of experts and weights that sum to one", rule);
   if (n_tokens == 0) return 0;
   const dim3 grid((n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), block(ROUTE_WARPS * 32);
   const size_t smem = (size_t)ROUTE_WARPS * 3 * E * sizeof(float);
@@ -570,8 +589,8 @@ extern "C" int bt_moe_route(const void* x, long long x_row_stride, const void* r
   };
 #define BT_ROUTE(T, NP)                                                                                              \
   BT_PDL_OK("moe_route", launch_pdl(moe_route_kernel<T, NP>, grid, block, smem, stream, 1, (const T*)x, x_row_stride, \
-                                    (const T*)router, n_tokens, K, E, top, n_groups, keep, scale, softmax, choice_bias, \
-                                    normalise, ids, weights))
+                                    (const T*)router, n_tokens, K, E, top, n_groups, keep, scale, rule, logit_bias, \
+                                    choice_bias, normalise, ids, weights))
   if (dtype == kF32) {
     const int np = pieces_of(4);
     if (np == 1) BT_ROUTE(float, 1); else if (np == 2) BT_ROUTE(float, 2); else if (np == 4) BT_ROUTE(float, 4);

@@ -16,8 +16,9 @@ from .errors import KernelError, ShapeError
 _LIB = None
 DTYPE_CODE = {torch.float32: 0, torch.bfloat16: 1}
 ACTIVATIONS = {None: 0, "none": 0, "gelu_new": 1, "gelu_tanh": 1, "gelu": 2, "gelu_erf": 2}
-# rules for the (gate, up) pair of a gated feed-forward: the activations above on the gate, or the clamped rule
-PAIR_RULES = dict(ACTIVATIONS, swish_clamp=3)
+# rules for the (gate, up) pair of a gated feed-forward: the activations above or x sigmoid(x) on the gate, or the clamped
+# rule
+PAIR_RULES = dict(ACTIVATIONS, swish_clamp=3, swish=4)
 PAGE_SIZE = 64
 
 
@@ -946,18 +947,25 @@ def mlstm_scan_fuses(dim: int, vdim: int) -> bool:
     return bool(library().bt_mlstm_scan_fuses(c_int(dim), c_int(vdim)))
 
 
+ROUTER_RULES = {"sigmoid": 0, "softmax": 1, "softmax_of_chosen": 2}
+
+
 def moe_route(x, router, ids, weights, *, n_tokens, top, n_groups=1, keep=1, scale=1.0, rule="sigmoid", choice_bias=None,
-              normalise=True):
+              normalise=True, logit_bias=None):
     """Per token the `top` experts with the largest sigmoid(router x) among the experts of the `keep` best of `n_groups`
     groups of neighbours (a group's score: the sum of its two largest), and their weights score / (sum + 1e-20) * scale.
     x [tokens, K] and router [experts, K] in the compute type, the products summed in 32-bit; ids int32 and weights
     32-bit, [tokens, top].  `rule` "softmax": the scores are softmax(router x) over all experts.  `choice_bias` [experts]
-    (32-bit) is added to the scores for the choice only; without `normalise` a weight is the chosen score as it is."""
+    (32-bit) is added to the scores for the choice only; without `normalise` a weight is the chosen score as it is.
+    `logit_bias` [experts] (32-bit) is added to router x.  `rule` "softmax_of_chosen": the experts with the largest router
+    x, weighted by the softmax over those, times scale."""
     e, k = router.shape
-    if rule not in ("sigmoid", "softmax"):
+    if rule not in ROUTER_RULES:
         raise ShapeError(f"moe_route: unknown rule {rule!r}")
     if choice_bias is not None:
         _need(choice_bias, "choice_bias", torch.float32, (e,))
+    if logit_bias is not None:
+        _need(logit_bias, "logit_bias", torch.float32, (e,))
     _need(x, "x", (torch.float32, torch.bfloat16), (None, k))
     _need(router, "router", x.dtype)
     _need(ids, "ids", torch.int32, (None, top))
@@ -967,7 +975,8 @@ def moe_route(x, router, ids, weights, *, n_tokens, top, n_groups=1, keep=1, sca
     _work(2.0 * n_tokens * e * k, n_tokens * k * x.element_size())
     _check(library().bt_moe_route(_ptr(x), c_longlong(x.stride(0)), _ptr(router), c_int(n_tokens), c_int(k), c_int(e),
                                   c_int(top), c_int(n_groups), c_int(keep), c_float(scale),
-                                  c_int(1 if rule == "softmax" else 0), _ptr(choice_bias), c_int(1 if normalise else 0),
+                                  c_int(ROUTER_RULES[rule]), _ptr(logit_bias), _ptr(choice_bias),
+                                  c_int(1 if normalise else 0),
                                   _ptr(ids), _ptr(weights), c_int(_code(x.dtype)), _stream()))
 
 
@@ -1384,6 +1393,29 @@ def selective_scan(x, z, dt, low, b_off, c_off, a_log, d_skip, state, slots, seq
                                        c_int(n_seqs), c_int(channels), c_int(n_state), c_float(out_scale), c_int(piece),
                                        c_int(max_pieces), _ptr(scratch) if piece else c_void_p(0),
                                        c_int(_code(x.dtype)), _stream()))
+
+
+# ---- the gated average of a minimal GRU --------------------------------------------------------------------------------
+
+def min_gru(proj, z_off, x_off, g_off, z_bias, x_bias, state, slots, seq_start, out, *, n_seqs, max_new):
+    """S <- (1 - z) S + z v, out = S * g sigmoid(g) per channel over the step's tokens of every sequence, with z = sigmoid(a +
+    z_bias), v = u + 1/2 for u >= 0 and sigmoid(u) below, u = x + x_bias (csrc/min_gru.cu).  a, x and g are the channels
+    `z_off`.., `x_off`.. and `g_off`.. of the rows of `proj`; state [slots, width] 32-bit, read and written at
+    `slots[seq]`; out: view [tokens, width] of proj's type.  No sequence brings more than `max_new` tokens."""
+    width = state.shape[1]
+    _need(proj, "proj", (torch.float32, torch.bfloat16))
+    _need(state, "state", torch.float32, (None, width))
+    _need(z_bias, "z_bias", torch.float32, (width,))
+    _need(x_bias, "x_bias", torch.float32, (width,))
+    _channels_view(out, "min_gru: out", 0, width)
+    if out.dtype != proj.dtype or min(z_off, x_off, g_off) < 0 or max(z_off, x_off, g_off) + width > proj.shape[1]:
+        raise ShapeError("min_gru: out has proj's type, and the three runs of channels lie inside its rows")
+    rows = out.shape[0]
+    _work(0.0, rows * width * 4.0 * proj.element_size() + 8.0 * n_seqs * width)
+    _check(library().bt_min_gru(_ptr(proj), c_longlong(proj.shape[1]), c_int(z_off), c_int(x_off), c_int(g_off),
+                                _ptr(z_bias), _ptr(x_bias), _ptr(state), _ptr(slots), _ptr(seq_start), _ptr(out),
+                                c_longlong(out.stride(0)), c_int(n_seqs), c_int(width), c_int(max_new),
+                                c_int(_code(proj.dtype)), _stream()))
 
 
 # ---- token shift, sigmoid attention -----------------------------------------------------------------------------------

@@ -4,3 +4,4 @@ from . import sovozen  # noqa: F401
 from . import gokezen  # noqa: F401
 from . import rakarax  # noqa: F401
 from . import bosalix  # noqa: F401
+from . import visadra  # noqa: F401

@@ -7,6 +7,7 @@ from .feed_forward import DenseFeedForward, GatedFeedForward, PolyNormFeedForwar
 from .latent_attention import LatentAttention
 from .lightning import LightningAttention, Retention
 from .matrix_memory import MatrixMemory
+from .min_gru import MinGru
 from .norm import LayerNorm, RmsNorm
 from .routed import RoutedFeedForward
 from .selective_scan import SelectiveScan
@@ -20,4 +21,4 @@ __all__ = ["CausalSelfAttention", "Block", "FeedForward", "Mixer", "Norm", "Part
            "LightningAttention", "MatrixMemory", "ParallelBlock", "RoutedFeedForward", "SideBySideMixers",
            "LayerNorm", "RmsNorm", "InterleavedRotary", "LearnedPositions", "NoPositions", "SandwichBlock",
            "TalkingConvAttention", "PolyNormFeedForward", "Retention", "SelectiveScan", "HalfSplitRotary", "OutputNormBlock",
-           "SigmoidAttention", "TokenShift"]
+           "SigmoidAttention", "TokenShift", "MinGru"]

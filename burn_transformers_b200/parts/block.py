@@ -230,6 +230,8 @@ class OutputNormBlock(Block):
             found["shift"] = self.shift
         if self.feed_forward is not None:
             found.update({"feed_forward": self.feed_forward, "norm2": self.norm2})
+            for name, part in getattr(self.feed_forward, "parts", dict)().items():
+                found["feed_forward." + name] = part
         return found
 
     def cache_need(self):
@@ -277,7 +279,7 @@ class OutputNormBlock(Block):
                             next_out=None if exact else rows)
         x = residual if exact else rows
         more = {"x32": residual} if getattr(self.feed_forward, "wants_x32", False) else {}
-        if getattr(self.feed_forward, "can_store", False) and getattr(self.feed_forward, "shared", None) is None:
+        if getattr(self.feed_forward, "can_store", False):
             self.feed_forward.forward(ctx, x, branch, store=True, **more)
         else:
             branch.zero_()

@@ -7,8 +7,8 @@ from .base import FeedForward
 from .linear import linear
 
 ACTIVATIONS = ("gelu_new", "gelu")
-# rules for the (gate, up) pair of a gated feed-forward: an activation on the gate, or the clamped rule
-PAIR_RULES = ACTIVATIONS + ("swish_clamp",)
+# rules for the (gate, up) pair of a gated feed-forward: an activation or x sigmoid(x) on the gate, or the clamped rule
+PAIR_RULES = ACTIVATIONS + ("swish_clamp", "swish")
 
 
 class DenseFeedForward(FeedForward):
@@ -47,11 +47,13 @@ class DenseFeedForward(FeedForward):
 class GatedFeedForward(FeedForward):
     """down(act(gate(x)) * up(x)), added to the residual stream; no biases.  The gate and up matrices are one product:
     `gate_up.weight` is [2 * inner, width] (stored [out, in]: the gate's rows, then up's), `down.weight` [width, inner].
-    The activation and the product of the two halves are formed in 32-bit and rounded once.  With the rule
+    The activation (`swish`: x sigmoid(x)) and the product of the two halves are formed in 32-bit and rounded once.  With the rule
     `swish_clamp` the hidden row is g' sigmoid(1.702 g') (u' + 1), g' = min(gate x, limit), u' = up x clamped to
     [-limit, limit]."""
 
     accepts_lazy_norm = True
+    # `forward(..., store=True)` writes the result into `residual` instead of adding it (rows that hold nothing yet)
+    can_store = True
 
     def __init__(self, width: int, inner: int, activation: str = "gelu_new", *, limit: float = 0.0,
                  init_std: float = 0.02, down_init_std: float | None = None):
@@ -65,7 +67,7 @@ class GatedFeedForward(FeedForward):
         return {"gate_up.weight": TensorSpec((2 * self.inner, self.width), MATRIX, ("normal", self.init_std)),
                 "down.weight": TensorSpec((self.width, self.inner), MATRIX, ("normal", self.down_init_std))}
 
-    def forward(self, ctx, x, residual):
+    def forward(self, ctx, x, residual, store=False):
         if getattr(ctx, "program", None) is not None:
             from ..engine.program import ProgramUnsupported
             raise ProgramUnsupported("a gated feed-forward has no phase in the fused step")
@@ -75,7 +77,7 @@ class GatedFeedForward(FeedForward):
         linear(ctx, x, self.t_gate_up_weight, None, both, m=n, w_is_nk=True)
         hidden = ctx.ws.take((n, self.inner), ctx.dtype)
         kernels.gated_activation(both, hidden, n_rows=n, activation=self.activation, limit=self.limit)
-        linear(ctx, hidden, self.t_down_weight, None, residual, m=n, residual=residual, w_is_nk=True)
+        linear(ctx, hidden, self.t_down_weight, None, residual, m=n, residual=None if store else residual, w_is_nk=True)
         ctx.ws.release(mark)
 
 

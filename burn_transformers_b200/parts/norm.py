@@ -41,19 +41,24 @@ class LayerNorm(Norm):
 
 class RmsNorm(Norm):
     """x / sqrt(mean(x^2) + eps) * (offset + weight) over the last axis, in 32-bit, eps inside the root; no shift.
-    `offset` 1: the file keeps the gain minus one; the sum is formed once, in 32-bit, when the weights are bound."""
+    `offset` 1: the file keeps the gain minus one; the sum is formed once, in 32-bit, when the weights are bound.
+    `one_gain`: the file keeps a single number (a tensor of no axes) that scales all channels; it is spread over the
+    channels when the weights are bound, so that every kernel that takes a norm's weight takes this one."""
 
     has_bias = False
 
-    def __init__(self, width: int, eps: float, offset: float = 0.0):
-        self.width, self.eps, self.offset = width, float(eps), float(offset)
+    def __init__(self, width: int, eps: float, offset: float = 0.0, one_gain: bool = False):
+        self.width, self.eps, self.offset, self.one_gain = width, float(eps), float(offset), one_gain
 
     def specs(self):
-        return {"weight": TensorSpec((self.width,), VECTOR, ("ones",) if self.offset == 0.0 else ("normal", 0.1))}
+        shape = () if self.one_gain else (self.width,)
+        return {"weight": TensorSpec(shape, VECTOR, ("ones",) if self.offset == 0.0 else ("normal", 0.1))}
 
     def bind(self, tensors):
         if self.offset != 0.0:
             tensors = {name: t.to(torch.float32) + self.offset for name, t in tensors.items()}
+        if self.one_gain:
+            tensors = {name: t.to(torch.float32).reshape(1).expand(self.width).contiguous() for name, t in tensors.items()}
         super().bind(tensors)
 
     def forward(self, ctx, x32, out_dtype, rows=None, n_rows=None, lazy=False):

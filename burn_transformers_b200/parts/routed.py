@@ -28,11 +28,14 @@ class RoutedFeedForward(FeedForward):
         router="softmax"     s = softmax(W_r h) over all experts
         choice_bias=True     the experts are chosen by s + `router.correction`; the weights still come from s
         normalise=False      weight_e = s_e, the chosen scores as they are
+        router="softmax_of_chosen"   s = W_r h; the weights are the softmax over the chosen s, times scale
+        logit_bias=True      `router.bias` is added to W_r h in 32-bit
         identity=k           the router has k more outputs, experts without tensors whose result is their input: a
                              token that chooses one gets weight_e * h (h in 32-bit: `forward(..., x32=)`)
         gated=False          an expert is down_e(act(up_e h)) with `activation` one of kernels.ACTIVATIONS
 
     Tensors: `router.weight` [experts + identity, width]; `router.correction` [experts + identity] (with `choice_bias`);
+    `router.bias` [experts + identity] (with `logit_bias`);
     `in.weight` [experts * 2 * inner, width] (per expert the gate's rows, then up's; without a gate [experts * inner,
     width]); `out.weight` [experts * width, inner].  `shared` is a feed-forward part of its own.
     """
@@ -42,12 +45,16 @@ class RoutedFeedForward(FeedForward):
     def __init__(self, width: int, n_experts: int, top: int, inner: int, *, activation: str = "swish_clamp",
                  limit: float = 0.0, n_groups: int = 1, keep: int = 1, scale: float = 1.0, shared: FeedForward | None = None,
                  init_std: float = 0.02, down_init_std: float | None = None, router: str = "sigmoid",
-                 choice_bias: bool = False, normalise: bool = True, identity: int = 0, gated: bool = True):
+                 choice_bias: bool = False, normalise: bool = True, identity: int = 0, gated: bool = True,
+                 logit_bias: bool = False):
         if min(width, n_experts, top, inner, n_groups, keep) <= 0:
             raise ShapeError("routed feed-forward: sizes must be positive")
-        if identity < 0 or (identity and n_groups != 1) or router not in ("sigmoid", "softmax"):
+        if identity < 0 or (identity and n_groups != 1) or router not in kernels.ROUTER_RULES:
             raise ShapeError("routed feed-forward: experts without tensors go with one group of experts; the router is "
-                             "`sigmoid` or `softmax`")
+                             f"one of {sorted(kernels.ROUTER_RULES)}")
+        if router == "softmax_of_chosen" and (n_groups != 1 or not normalise):
+            raise ShapeError("routed feed-forward: a softmax over the chosen experts goes with one group of experts and "
+                             "weights that sum to one")
         if (n_experts + identity) % n_groups or keep > n_groups or top > keep * ((n_experts + identity) // n_groups):
             raise ShapeError(f"routed feed-forward: {n_experts} experts in {n_groups} groups of which {keep} are kept "
                              f"cannot give {top} experts a token")
@@ -59,6 +66,7 @@ class RoutedFeedForward(FeedForward):
         self.activation, self.limit = activation, float(limit)
         self.n_groups, self.keep, self.scale, self.shared = n_groups, keep, float(scale), shared
         self.router, self.has_choice_bias, self.normalise = router, choice_bias, normalise
+        self.has_logit_bias = logit_bias
         self.identity, self.gated = int(identity), gated
         self.in_rows = (2 if gated else 1) * inner          # rows of an expert's first matrix
         self.init_std = init_std
@@ -71,6 +79,8 @@ class RoutedFeedForward(FeedForward):
                  "out.weight": TensorSpec((e * self.width, self.inner), MATRIX, ("normal", self.down_init_std))}
         if self.has_choice_bias:
             specs["router.correction"] = TensorSpec((routes,), VECTOR, ("normal", 0.05))
+        if self.has_logit_bias:
+            specs["router.bias"] = TensorSpec((routes,), VECTOR, ("normal", 0.1))
         return specs
 
     def parts(self):
@@ -115,7 +125,8 @@ class RoutedFeedForward(FeedForward):
         weights = ctx.ws.take((n, top), torch.float32)
         kernels.moe_route(x, self.t_router_weight, ids, weights, n_tokens=n, top=top, n_groups=self.n_groups,
                           keep=self.keep, scale=self.scale, rule=self.router,
-                          choice_bias=self.t_router_correction if self.has_choice_bias else None, normalise=self.normalise)
+                          choice_bias=self.t_router_correction if self.has_choice_bias else None, normalise=self.normalise,
+                          logit_bias=self.t_router_bias if self.has_logit_bias else None)
         # (the pairs of experts without tensors sort behind the others' rows, where no product looks)
         offsets = ctx.ws.take((routes + 1,), torch.int32)
         tile_first = ctx.ws.take((routes + 1,), torch.int32)
