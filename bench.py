@@ -1,7 +1,7 @@
 """Decode and prefill throughput of GPT-2 (random weights, synthetic tokens) on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--points all|small] [--profile]
-    python bench.py --arch sovozen|gokezen|rakarax|bosalix [--sizes small,medium]
+    python bench.py --arch sovozen|gokezen|rakarax|bosalix|visadra [--sizes small,medium]
 
 A step is one decode step of a batch of 8 sequences of GPT-2 small.  The run prints one JSON line: `value` is decoded
 tokens per second, timed on the device with CUDA events over exactly K steps; `e2e` is the same through the public
@@ -441,14 +441,35 @@ def bosalix(size: str) -> dict:
             "embedding": {"scale": 1.0}, "layers": [dict(latent) if i % 2 else dict(sigmoid) for i in range(n_layer)]}
 
 
+def visadra(size: str) -> dict:
+    """A Visadra with as many layers, the width and the heads of GPT-2 `size`: in turn a minimal GRU with a dense
+    feed-forward, a latent attention (latent 256 or 512 + 32 or 64 rotated, a sink) with routed experts (16, 4 a token,
+    and a shared one), a minimal GRU with routed experts, a latent attention with a dense feed-forward; the GRUs as wide
+    as the model, every feed-forward with the weights a token uses equal to GPT-2's (3 x ff x width = 8 x width^2)."""
+    n_layer, width, heads = {"small": (12, 768, 12), "medium": (24, 1024, 16)}[size]
+    rank, rot = {"small": (256, 32), "medium": (512, 64)}[size]
+    ff, expert_ff, shared_ff = {"small": (2048, 384, 512), "medium": (2816, 512, 768)}[size]
+    dim = 64
+    dense = {"kind": "dense", "ff": ff}
+    routed = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": 16, "top": 4}, "shared": {"ff": shared_ff}}
+    latent = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": dim, "kv_rank": rank, "scale": (dim + rot) ** -0.5,
+              "rot": {"dims": rot, "base": 10000.0}}
+    kinds = [("mingru", {"width": width}, dense), ("latent_attention", latent, routed), ("mingru_2", {"width": width}, routed),
+             ("latent_attention", latent, dense)]
+    layers = [{"type": kind, "mixer": mixer, "mlp": mlp} for kind, mixer, mlp in (kinds[i % 4] for i in range(n_layer))]
+    return {"architecture": "Visadra", "vocab": 50257, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "logit_scale": 1.0, "layers": layers}
+
+
 ARCH_PAIRS = {"sovozen": (sovozen, "gpt2", gpt2), "gokezen": (gokezen, "sovozen", sovozen),
-              "rakarax": (rakarax, "gokezen", gokezen), "bosalix": (bosalix, "gokezen", gokezen)}
+              "rakarax": (rakarax, "gokezen", gokezen), "bosalix": (bosalix, "gokezen", gokezen),
+              "visadra": (visadra, "bosalix", bosalix)}
 
 
 def run_arch_compare(args):
-    """--arch sovozen | gokezen | rakarax | bosalix: prefill and decode throughput of that design beside the library's
+    """--arch sovozen | gokezen | rakarax | bosalix | visadra: prefill and decode throughput of that design beside the library's
     closest other model at the same width and depth (GPT-2 for Sovozen, Sovozen for Gokezen, Gokezen for Rakarax and for
-    Bosalix; random weights, bfloat16), and where each
+    Bosalix, Bosalix for Visadra; random weights, bfloat16), and where each
     spends a prefill and a decode step, kernel by kernel, against the measured peaks.  One JSON line; the default
     workload of this file is untouched."""
     import numpy as np
@@ -669,10 +690,10 @@ def main() -> int:
     parser.add_argument("--profile", action="store_true",
                         help="print where a prefill and a decode step spend their time, kernel by kernel, instead")
     parser.add_argument("--model", choices=["small", "medium", "xl"], default="small", help="the model --profile looks at")
-    parser.add_argument("--arch", choices=["gpt2", "sovozen", "gokezen", "rakarax", "bosalix"], default="gpt2",
-                        help="sovozen, gokezen, rakarax, bosalix: measure that design beside the closest other model of equal width and "
+    parser.add_argument("--arch", choices=["gpt2", "sovozen", "gokezen", "rakarax", "bosalix", "visadra"], default="gpt2",
+                        help="sovozen, gokezen, rakarax, bosalix, visadra: measure that design beside the closest other model of equal width and "
                              "depth instead (see --sizes)")
-    parser.add_argument("--sizes", default="small,medium", help="with --arch sovozen | gokezen | rakarax | bosalix: which widths (small, medium)")
+    parser.add_argument("--sizes", default="small,medium", help="with an --arch other than gpt2: which widths (small, medium)")
     args = parser.parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable": "the reference is a Rust crate (Cargo.toml only): pip "
