@@ -136,8 +136,9 @@ int bt_lightning_chunked(const void* proj, long long row_stride, int q_off, int 
 int bt_rmsnorm(const void* x, int x_dtype, long long x_row_stride, const float* weight, const void* gate, int gate_dtype,
                long long gate_row_stride, void* out, int out_dtype, long long out_row_stride, int n_rows, int width,
                int groups, float eps, int gate_rule, cudaStream_t stream);
-int bt_rmsnorm_add(const float* x, const float* weight, float* stream_rows, const float* next_weight, void* next_out,
-                   int next_dtype, long long n_rows, int width, float eps, float factor, cudaStream_t stream);
+int bt_rmsnorm_add(const float* x, const int* place, int top, const float* extra, const float* weight, float* stream_rows,
+                   const float* next_weight, void* next_out, int next_dtype, long long n_rows, int width, float eps,
+                   float factor, cudaStream_t stream);
 // The blend of every row with the row of the token before it, with the kept row per sequence (csrc/rowwise.cu).
 int bt_token_shift(const float* x, const float* shift, float* state, const int* slots, const int* seq_start,
                    const int* token_seq, void* out, int out_dtype, long long n_rows, int width, cudaStream_t stream);

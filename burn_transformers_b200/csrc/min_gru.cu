@@ -23,7 +23,7 @@ namespace bt {
 
 namespace cg = cooperative_groups;
 
-constexpr int MG_WARPS = 16, MG_TOK = 8, MG_MAX_CLUSTER = 8;
+constexpr int MG_WARPS = 8, MG_TOK = 8, MG_MAX_CLUSTER = 8, MG_BLOCKS = 2;
 constexpr int MG_FEW = 16;       // runs of at most this many tokens are walked by single threads
 
 struct MinGruArgs {
@@ -40,196 +40,220 @@ struct MinGruArgs {
   int width;
 };
 
-__device__ __forceinline__ float logistic(float v) { return 1.f / (1.f + expf(-v)); }
+// 32-bit rows take CUDA's full-precision functions; rows that come as bfloat16 (and leave rounded to it) the
+// special-function unit's exponential and reciprocal, whose errors are a few units in the last place of 32-bit.
+template <bool EXACT> __device__ __forceinline__ float exponential(float v) { return EXACT ? expf(v) : __expf(v); }
+template <bool EXACT> __device__ __forceinline__ float quotient(float a, float b) { return EXACT ? a / b : __fdividef(a, b); }
+// (exp(-v) may overflow to infinity: the quotient is then zero, which is the limit)
+template <bool EXACT> __device__ __forceinline__ float logistic(float v) {
+  return quotient<EXACT>(1.f, 1.f + exponential<EXACT>(-v));
+}
 
 // the map of one token: keep = 1 - z, add = z * v.  With e = exp(-|s|), z and 1 - z are 1 / (1 + e) and e / (1 + e), one
 // or the other way round by the sign of s: neither is a difference of nearly equal numbers.
+template <bool EXACT>
 __device__ __forceinline__ void token_map(float s, float u, float& keep, float& add) {
-  const float e = expf(-fabsf(s)), big = 1.f / (1.f + e), small = e * big;
+  const float e = exponential<EXACT>(-fabsf(s)), big = quotient<EXACT>(1.f, 1.f + e), small = e * big;
   keep = s >= 0.f ? small : big;
   const float share = s >= 0.f ? big : small;
-  add = share * (u >= 0.f ? u + 0.5f : logistic(u));
+  add = share * (u >= 0.f ? u + 0.5f : logistic<EXACT>(u));
 }
 
-// V neighbouring channels as one access (V * sizeof(T) bytes; the host has checked the alignment)
-template <typename T, int V>
-__device__ __forceinline__ void load_channels(const T* p, float (&o)[V]) {
-  if constexpr (V == 1) {
-    o[0] = to_float(p[0]);
-  } else if constexpr (sizeof(T) == 4) {
-    const float2 f = *reinterpret_cast<const float2*>(p);
-    o[0] = f.x; o[1] = f.y;
-  } else {
-    const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
-    o[0] = f.x; o[1] = f.y;
-  }
+// V neighbouring channels as one access (V * sizeof(T) bytes; the host has checked the alignment), as they lie in memory
+template <typename T, int V> struct Raw;
+template <> struct Raw<float, 1> { float v; };
+template <> struct Raw<float, 2> { float2 v; };
+template <> struct Raw<__nv_bfloat16, 1> { __nv_bfloat16 v; };
+template <> struct Raw<__nv_bfloat16, 2> { __nv_bfloat162 v; };
+
+template <typename T, int V> __device__ __forceinline__ Raw<T, V> load_raw(const T* p) {
+  return *reinterpret_cast<const Raw<T, V>*>(p);
 }
-template <typename T, int V>
-__device__ __forceinline__ void store_channels(T* p, const float (&o)[V]) {
-  if constexpr (V == 1) {
-    p[0] = from_float<T>(o[0]);
-  } else if constexpr (sizeof(T) == 4) {
-    *reinterpret_cast<float2*>(p) = make_float2(o[0], o[1]);
-  } else {
-    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(o[0], o[1]);
-  }
+__device__ __forceinline__ void unpack(const Raw<float, 1>& r, float (&o)[1]) { o[0] = r.v; }
+__device__ __forceinline__ void unpack(const Raw<float, 2>& r, float (&o)[2]) { o[0] = r.v.x; o[1] = r.v.y; }
+__device__ __forceinline__ void unpack(const Raw<__nv_bfloat16, 1>& r, float (&o)[1]) { o[0] = __bfloat162float(r.v); }
+__device__ __forceinline__ void unpack(const Raw<__nv_bfloat16, 2>& r, float (&o)[2]) {
+  const float2 f = __bfloat1622float2(r.v);
+  o[0] = f.x; o[1] = f.y;
+}
+__device__ __forceinline__ void store_channels(float* p, const float (&o)[1]) { p[0] = o[0]; }
+__device__ __forceinline__ void store_channels(float* p, const float (&o)[2]) {
+  *reinterpret_cast<float2*>(p) = make_float2(o[0], o[1]);
+}
+__device__ __forceinline__ void store_channels(__nv_bfloat16* p, const float (&o)[1]) { p[0] = __float2bfloat16_rn(o[0]); }
+__device__ __forceinline__ void store_channels(__nv_bfloat16* p, const float (&o)[2]) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(o[0], o[1]);
 }
 
 template <typename T, int V>
 __global__ void __launch_bounds__(64) min_gru_few_kernel(MinGruArgs p) {
   const int c = (blockIdx.x * 64 + threadIdx.x) * V, seq = blockIdx.y;
-  float zb[V], xb[V];
+  constexpr bool EXACT = sizeof(T) == 4;
   const bool in = c < p.width;
-  if (in) { load_channels<float, V>(p.z_bias + c, zb); load_channels<float, V>(p.x_bias + c, xb); }
+  float zb[V], xb[V];
+  unpack(load_raw<float, V>(p.z_bias + (in ? c : 0)), zb);
+  unpack(load_raw<float, V>(p.x_bias + (in ? c : 0)), xb);
   pdl_trigger();
   pdl_wait();
   if (!in) return;
   const int first = p.seq_start[seq], last = p.seq_start[seq + 1];
   float* kept = p.state + (long long)p.slots[seq] * p.width + c;
   float s[V];
-  load_channels<float, V>(kept, s);
+  unpack(load_raw<float, V>(kept), s);
   const T* row = reinterpret_cast<const T*>(p.proj) + (long long)first * p.row_stride + c;
   T* out = reinterpret_cast<T*>(p.out) + (long long)first * p.out_stride + c;
   for (int t = first; t < last; ++t, row += p.row_stride, out += p.out_stride) {
     float a[V], x[V], g[V], y[V];
-    load_channels<T, V>(row + p.z_off, a);
-    load_channels<T, V>(row + p.x_off, x);
-    load_channels<T, V>(row + p.g_off, g);
+    const Raw<T, V> ra = load_raw<T, V>(row + p.z_off), rx = load_raw<T, V>(row + p.x_off), rg = load_raw<T, V>(row + p.g_off);
+    unpack(ra, a);
+    unpack(rx, x);
+    unpack(rg, g);
 #pragma unroll
     for (int i = 0; i < V; ++i) {
       float keep, add;
-      token_map(a[i] + zb[i], x[i] + xb[i], keep, add);
+      token_map<EXACT>(a[i] + zb[i], x[i] + xb[i], keep, add);
       s[i] = fmaf(keep, s[i], add);
-      y[i] = s[i] * (g[i] * logistic(g[i]));
+      y[i] = s[i] * (g[i] * logistic<EXACT>(g[i]));
     }
-    store_channels<T, V>(out, y);
+    store_channels(out, y);
   }
-  store_channels<float, V>(kept, s);
+  store_channels(kept, s);
+}
+
+// The map S -> keep S + add of a run of tokens, for a lane's V channels.
+template <int V> struct __align__(8 * V) RunMap { float keep[V], add[V]; };
+
+template <int V> __device__ __forceinline__ void then(RunMap<V>& m, const RunMap<V>& next) {
+#pragma unroll
+  for (int i = 0; i < V; ++i) {
+    m.add[i] = fmaf(next.keep[i], m.add[i], next.add[i]);
+    m.keep[i] *= next.keep[i];
+  }
 }
 
 // grid (channel groups * cluster, sequences), cluster blocks along x; block: MG_WARPS warps.
 template <typename T, int V>
-__global__ void __launch_bounds__(MG_WARPS * 32)
+__global__ void __launch_bounds__(MG_WARPS * 32, MG_BLOCKS)
 min_gru_scan_kernel(MinGruArgs p, int cluster_size) {
   constexpr int CH = 32 * V;
-  __shared__ float warp_keep[MG_WARPS][CH], warp_add[MG_WARPS][CH];     // the warps' maps, then what comes before each
-  __shared__ float block_keep[2][CH], block_add[2][CH];                 // the block's map, by turns (peers read it)
-  __shared__ float enter[CH];                                           // the state before the block's first token
+  constexpr bool EXACT = sizeof(T) == 4;
+  __shared__ RunMap<V> warp_map[MG_WARPS][32];      // the warps' maps, then the map of all tokens before each warp's
+  __shared__ RunMap<V> block_map[2][32];            // the block's map, by turns (peers read it)
+  __shared__ float enter[32][V];                    // the state before the block's first token
   cg::cluster_group cluster = cg::this_cluster();
   const int rank = (int)cluster.block_rank();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int c = (blockIdx.x / cluster_size) * CH + lane * V, seq = blockIdx.y;
-  const bool in = c < p.width;
-  float zb[V] = {}, xb[V] = {};
-  if (in) { load_channels<float, V>(p.z_bias + c, zb); load_channels<float, V>(p.x_bias + c, xb); }
+  const int c0 = (blockIdx.x / cluster_size) * CH + lane * V, seq = blockIdx.y;
+  const bool in = c0 < p.width;
+  const int c = in ? c0 : 0;             // (a lane behind the last channel computes the first one's and stores nothing)
+  float zb[V], xb[V];
+  unpack(load_raw<float, V>(p.z_bias + c), zb);
+  unpack(load_raw<float, V>(p.x_bias + c), xb);
   pdl_trigger();
   pdl_wait();
   const int first = p.seq_start[seq], count = p.seq_start[seq + 1] - first;
   float* kept = p.state + (long long)p.slots[seq] * p.width + c;
   float s[V] = {};                       // (warp 0: the state before this round of the loop)
-  if (warp == 0 && in) load_channels<float, V>(kept, s);
+  if (warp == 0) unpack(load_raw<float, V>(kept), s);
   const T* rows = reinterpret_cast<const T*>(p.proj) + (long long)first * p.row_stride + c;
   T* outs = reinterpret_cast<T*>(p.out) + (long long)first * p.out_stride + c;
   const int round_tokens = cluster_size * MG_WARPS * MG_TOK;
+  // all reads of a warp's tokens in flight together: no branch, a place behind the run's last token reads that one
+  Raw<T, V> ra[MG_TOK], rx[MG_TOK], rg[MG_TOK];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int k = 0; k < MG_TOK; ++k) {
+      const T* row = rows + (long long)min(t0 + k, count - 1) * p.row_stride;
+      ra[k] = load_raw<T, V>(row + p.z_off);
+      rx[k] = load_raw<T, V>(row + p.x_off);
+      rg[k] = load_raw<T, V>(row + p.g_off);
+    }
+  };
+  const int mine = (rank * MG_WARPS + warp) * MG_TOK;
+  if (count > 0) fetch(mine);
   int turn = 0;
   for (int base = 0; base < count; base += round_tokens, turn ^= 1) {
-    const int t0 = base + (rank * MG_WARPS + warp) * MG_TOK;
-    float keep[MG_TOK][V], add[MG_TOK][V], g[MG_TOK][V];
-    {
-      float a[MG_TOK][V], x[MG_TOK][V];
+    const int t0 = base + mine;
+    float keep[MG_TOK][V], add[MG_TOK][V];
+    Raw<T, V> gate[MG_TOK];
 #pragma unroll
-      for (int k = 0; k < MG_TOK; ++k) {           // (all reads of the warp's tokens are in flight together)
-#pragma unroll
-        for (int i = 0; i < V; ++i) a[k][i] = x[k][i] = g[k][i] = 0.f;
-        if (in && t0 + k < count) {
-          const T* row = rows + (long long)(t0 + k) * p.row_stride;
-          load_channels<T, V>(row + p.z_off, a[k]);
-          load_channels<T, V>(row + p.x_off, x[k]);
-          load_channels<T, V>(row + p.g_off, g[k]);
-        }
-      }
-#pragma unroll
-      for (int k = 0; k < MG_TOK; ++k)
-#pragma unroll
-        for (int i = 0; i < V; ++i) {
-          keep[k][i] = 1.f;                        // (a place behind the run's last token leaves the state as it is)
-          add[k][i] = 0.f;
-          if (t0 + k < count) token_map(a[k][i] + zb[i], x[k][i] + xb[i], keep[k][i], add[k][i]);
-        }
-    }
-#pragma unroll
-    for (int i = 0; i < V; ++i) {
-      float ka = 1.f, ad = 0.f;
-#pragma unroll
-      for (int k = 0; k < MG_TOK; ++k) {
-        ad = fmaf(keep[k][i], ad, add[k][i]);
-        ka *= keep[k][i];
-      }
-      warp_keep[warp][lane * V + i] = ka;
-      warp_add[warp][lane * V + i] = ad;
-    }
-    __syncthreads();
-    if (warp == 0) {
+    for (int k = 0; k < MG_TOK; ++k) {
+      float a[V], x[V];
+      unpack(ra[k], a);
+      unpack(rx[k], x);
+      gate[k] = rg[k];
 #pragma unroll
       for (int i = 0; i < V; ++i) {
-        const int j = lane * V + i;
-        float ka = 1.f, ad = 0.f;
-#pragma unroll
-        for (int w = 0; w < MG_WARPS; ++w) {
-          const float wk = warp_keep[w][j], wa = warp_add[w][j];
-          warp_keep[w][j] = ka;
-          warp_add[w][j] = ad;
-          ad = fmaf(wk, ad, wa);
-          ka *= wk;
+        token_map<EXACT>(a[i] + zb[i], x[i] + xb[i], keep[k][i], add[k][i]);
+        if (t0 + k >= count) {                   // (... and leaves the state as it is)
+          keep[k][i] = 1.f;
+          add[k][i] = 0.f;
         }
-        block_keep[turn][j] = ka;
-        block_add[turn][j] = ad;
       }
+    }
+    if (base + round_tokens < count) fetch(t0 + round_tokens);      // (the next round's, while this one's maps meet)
+    RunMap<V> m;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      m.keep[i] = keep[0][i];
+      m.add[i] = add[0][i];
+#pragma unroll
+      for (int k = 1; k < MG_TOK; ++k) {
+        m.add[i] = fmaf(keep[k][i], m.add[i], add[k][i]);
+        m.keep[i] *= keep[k][i];
+      }
+    }
+    warp_map[warp][lane] = m;
+    __syncthreads();
+    if (warp == 0) {
+      RunMap<V> all = {};
+#pragma unroll
+      for (int i = 0; i < V; ++i) all.keep[i] = 1.f;
+#pragma unroll
+      for (int w = 0; w < MG_WARPS; ++w) {
+        const RunMap<V> own = warp_map[w][lane];
+        warp_map[w][lane] = all;
+        then(all, own);
+      }
+      block_map[turn][lane] = all;
     }
     cluster.sync();                    // every block's map is there (and, block by block, the warps' prefixes)
     if (warp == 0) {
-      float pk[MG_MAX_CLUSTER][V], pa[MG_MAX_CLUSTER][V];
+      RunMap<V> peer[MG_MAX_CLUSTER];
 #pragma unroll
-      for (int b = 0; b < MG_MAX_CLUSTER; ++b)
+      for (int b = 0; b < MG_MAX_CLUSTER; ++b) {
 #pragma unroll
-        for (int i = 0; i < V; ++i) {
-          pk[b][i] = 1.f;
-          pa[b][i] = 0.f;
-          if (b < cluster_size) {
-            pk[b][i] = cluster.map_shared_rank(&block_keep[turn][0], b)[lane * V + i];
-            pa[b][i] = cluster.map_shared_rank(&block_add[turn][0], b)[lane * V + i];
-          }
-        }
+        for (int i = 0; i < V; ++i) { peer[b].keep[i] = 1.f; peer[b].add[i] = 0.f; }
+        if (b < cluster_size) peer[b] = *cluster.map_shared_rank(&block_map[turn][lane], b);
+      }
 #pragma unroll
       for (int i = 0; i < V; ++i) {
 #pragma unroll
         for (int b = 0; b < MG_MAX_CLUSTER; ++b) {
-          if (b == rank) enter[lane * V + i] = s[i];
-          s[i] = fmaf(pk[b][i], s[i], pa[b][i]);
+          if (b == rank) enter[lane][i] = s[i];
+          s[i] = fmaf(peer[b].keep[i], s[i], peer[b].add[i]);
         }
       }
     }
     __syncthreads();
-    if (in) {
-      float y[V], st[V];
+    const RunMap<V> before = warp_map[warp][lane];
+    float st[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) st[i] = fmaf(before.keep[i], enter[lane][i], before.add[i]);
+#pragma unroll
+    for (int k = 0; k < MG_TOK; ++k) {
+      float g[V], y[V];
+      unpack(gate[k], g);
 #pragma unroll
       for (int i = 0; i < V; ++i) {
-        const int j = lane * V + i;
-        st[i] = fmaf(warp_keep[warp][j], enter[j], warp_add[warp][j]);
+        st[i] = fmaf(keep[k][i], st[i], add[k][i]);
+        y[i] = st[i] * (g[i] * logistic<EXACT>(g[i]));
       }
-#pragma unroll
-      for (int k = 0; k < MG_TOK; ++k) {
-#pragma unroll
-        for (int i = 0; i < V; ++i) {
-          st[i] = fmaf(keep[k][i], st[i], add[k][i]);
-          y[i] = st[i] * (g[k][i] * logistic(g[k][i]));
-        }
-        if (t0 + k < count) store_channels<T, V>(outs + (long long)(t0 + k) * p.out_stride, y);
-      }
+      if (in && t0 + k < count) store_channels(outs + (long long)(t0 + k) * p.out_stride, y);
     }
     __syncthreads();                   // (the next round writes the warps' maps and `enter` again)
   }
-  if (rank == 0 && warp == 0 && in) store_channels<float, V>(kept, s);
+  if (rank == 0 && warp == 0 && in) store_channels(kept, s);
   cluster.sync();                      // nobody leaves while a peer may still read its map
 }
 

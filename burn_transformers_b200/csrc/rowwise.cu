@@ -303,36 +303,174 @@ extern "C" int bt_add_rows(float* x, const float* a, const float* b, const float
 
 namespace bt {
 
-// stream_rows[r] += x[r] / sqrt(mean(x[r]^2) + eps) * weight: a sublayer's result, normed, joins the 32-bit stream.
+// stream_rows[r] += factor * v[r] / sqrt(mean(v[r]^2) + eps) * weight: a sublayer's result v, normed, joins the 32-bit
+// stream.  v[r] is x[r], or, with `place`, the sum of the `top` rows x[place[r * top + j]] in that order (what the experts a
+// token chose left in rows sorted by expert); `extra` [rows, width] is added to it (a shared expert's result).
 // With next_out the row that the stream then holds is normed once more (next_weight) into next_out: the norm that
-// opens the next sublayer, in the same pass over the row.
+// opens the next sublayer, in the same pass over the row; without next_weight it is written as it is.
+struct NormAddArgs {
+  const float* x;
+  const int* place;
+  int top;
+  const float* extra;
+  const float* weight;
+  float* stream_rows;
+  const float* next_weight;
+  void* next_out;
+  int width;
+  float eps, factor;
+};
+
+__device__ __forceinline__ float norm_add_value(const NormAddArgs& p, long long r, int c) {
+  float v;
+  if (p.place == nullptr) {
+    v = p.x[r * p.width + c];
+  } else {
+    v = 0.f;
+    for (int j = 0; j < p.top; ++j) v += p.x[(long long)p.place[r * p.top + j] * p.width + c];
+  }
+  return p.extra != nullptr ? v + p.extra[r * p.width + c] : v;
+}
+
 template <typename TOut>
-__global__ void __launch_bounds__(128)
-rmsnorm_add_kernel(const float* __restrict__ x, const float* __restrict__ weight, float* __restrict__ stream_rows,
-                   const float* __restrict__ next_weight, TOut* __restrict__ next_out, int width, float eps, float factor) {
+__global__ void __launch_bounds__(128) rmsnorm_add_kernel(NormAddArgs p) {
   __shared__ float scratch[33];
   pdl_trigger();
   pdl_wait();
   const long long r = blockIdx.x;
-  const float* src = x + r * width;
-  float* dst = stream_rows + r * width;
+  float* dst = p.stream_rows + r * p.width;
+  TOut* next_out = reinterpret_cast<TOut*>(p.next_out);
   float ss = 0.f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) ss = fmaf(src[c], src[c], ss);
-  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+  for (int c = threadIdx.x; c < p.width; c += blockDim.x) {
+    const float v = norm_add_value(p, r, c);
+    ss = fmaf(v, v, ss);
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
   float ss2 = 0.f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const float v = fmaf(factor, src[c] * inv * weight[c], dst[c]);
+  for (int c = threadIdx.x; c < p.width; c += blockDim.x) {
+    const float v = fmaf(p.factor, norm_add_value(p, r, c) * inv * p.weight[c], dst[c]);
     dst[c] = v;
     ss2 = fmaf(v, v, ss2);
   }
   if (next_out == nullptr) return;
-  if (next_weight == nullptr) {       // the next sublayer reads the new row as it is, in its own element type
-    for (int c = threadIdx.x; c < width; c += blockDim.x) next_out[r * width + c] = from_float<TOut>(dst[c]);
+  if (p.next_weight == nullptr) {       // the next sublayer reads the new row as it is, in its own element type
+    for (int c = threadIdx.x; c < p.width; c += blockDim.x) next_out[r * p.width + c] = from_float<TOut>(dst[c]);
     return;
   }
-  const float inv2 = 1.f / sqrtf(block_sum(ss2, scratch) / (float)width + eps);
-  for (int c = threadIdx.x; c < width; c += blockDim.x)       // (a thread reads back what it wrote itself)
-    next_out[r * width + c] = from_float<TOut>(dst[c] * inv2 * next_weight[c]);
+  const float inv2 = 1.f / sqrtf(block_sum(ss2, scratch) / (float)p.width + p.eps);
+  for (int c = threadIdx.x; c < p.width; c += blockDim.x)       // (a thread reads back what it wrote itself)
+    next_out[r * p.width + c] = from_float<TOut>(dst[c] * inv2 * p.next_weight[c]);
+}
+
+__device__ __forceinline__ void store_four(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_four(__nv_bfloat16* p, const float4& v) {
+  uint2 o;
+  *reinterpret_cast<__nv_bfloat162*>(&o.x) = __floats2bfloat162_rn(v.x, v.y);
+  *reinterpret_cast<__nv_bfloat162*>(&o.y) = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = o;
+}
+__device__ __forceinline__ float square_sum(const float4& v, float s) {
+  return fmaf(v.w, v.w, fmaf(v.z, v.z, fmaf(v.y, v.y, fmaf(v.x, v.x, s))));
+}
+__device__ __forceinline__ void add_four(float4& v, const float4& a) { v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w; }
+
+// The same for rows of whole 16-byte pieces, at most NV of them a thread: the row stays in registers, every operand is
+// read once, and all reads that do not wait for the sum are asked for before it.
+template <typename TOut, int NV>
+__global__ void __launch_bounds__(128) rmsnorm_add_vec_kernel(NormAddArgs p) {
+  __shared__ float scratch[33];
+  const int pieces = p.width / 4;
+  float4 w[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int q = threadIdx.x + 128 * i;
+    w[i] = q < pieces ? reinterpret_cast<const float4*>(p.weight)[q] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  pdl_trigger();
+  pdl_wait();
+  const long long r = blockIdx.x;
+  float4 v[NV], d[NV];
+  float4* dst = reinterpret_cast<float4*>(p.stream_rows + r * p.width);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int q = threadIdx.x + 128 * i;
+    v[i] = d[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (q < pieces) d[i] = dst[q];
+  }
+  if (p.place == nullptr) {
+    const float4* src = reinterpret_cast<const float4*>(p.x + r * p.width);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int q = threadIdx.x + 128 * i;
+      if (q < pieces) v[i] = src[q];
+    }
+  } else {
+#pragma unroll 4
+    for (int j = 0; j < p.top; ++j) {
+      const float4* src = reinterpret_cast<const float4*>(p.x + (long long)p.place[r * p.top + j] * p.width);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int q = threadIdx.x + 128 * i;
+        if (q < pieces) add_four(v[i], src[q]);
+      }
+    }
+  }
+  if (p.extra != nullptr) {
+    const float4* src = reinterpret_cast<const float4*>(p.extra + r * p.width);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int q = threadIdx.x + 128 * i;
+      if (q < pieces) add_four(v[i], src[q]);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) ss = square_sum(v[i], ss);
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
+  float ss2 = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    d[i].x = fmaf(p.factor, v[i].x * inv * w[i].x, d[i].x);
+    d[i].y = fmaf(p.factor, v[i].y * inv * w[i].y, d[i].y);
+    d[i].z = fmaf(p.factor, v[i].z * inv * w[i].z, d[i].z);
+    d[i].w = fmaf(p.factor, v[i].w * inv * w[i].w, d[i].w);
+    ss2 = square_sum(d[i], ss2);
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int q = threadIdx.x + 128 * i;
+    if (q < pieces) dst[q] = d[i];
+  }
+  if (p.next_out == nullptr) return;
+  TOut* next = reinterpret_cast<TOut*>(p.next_out) + r * p.width;
+  const float inv2 = p.next_weight != nullptr ? 1.f / sqrtf(block_sum(ss2, scratch) / (float)p.width + p.eps) : 1.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int q = threadIdx.x + 128 * i;
+    if (q >= pieces) continue;
+    if (p.next_weight != nullptr) {
+      const float4 nw = reinterpret_cast<const float4*>(p.next_weight)[q];
+      d[i] = make_float4(d[i].x * inv2 * nw.x, d[i].y * inv2 * nw.y, d[i].z * inv2 * nw.z, d[i].w * inv2 * nw.w);
+    }
+    store_four(next + 4 * q, d[i]);
+  }
+}
+
+template <typename TOut>
+static int launch_norm_add(const NormAddArgs& p, long long n_rows, cudaStream_t stream) {
+  auto at16 = [](const void* ptr) { return (unsigned long long)ptr % 16 == 0; };
+  const dim3 grid((unsigned)n_rows), block(128);
+  const int pieces = p.width / 4;
+  if (p.width % 4 == 0 && pieces <= 8 * 128 && at16(p.x) && at16(p.extra) && at16(p.weight) && at16(p.stream_rows) &&
+      at16(p.next_weight) && at16(p.next_out)) {
+    if (pieces <= 128) BT_PDL_OK("rmsnorm_add", launch_pdl(rmsnorm_add_vec_kernel<TOut, 1>, grid, block, 0, stream, 1, p));
+    else if (pieces <= 256) BT_PDL_OK("rmsnorm_add", launch_pdl(rmsnorm_add_vec_kernel<TOut, 2>, grid, block, 0, stream, 1, p));
+    else if (pieces <= 512) BT_PDL_OK("rmsnorm_add", launch_pdl(rmsnorm_add_vec_kernel<TOut, 4>, grid, block, 0, stream, 1, p));
+    else BT_PDL_OK("rmsnorm_add", launch_pdl(rmsnorm_add_vec_kernel<TOut, 8>, grid, block, 0, stream, 1, p));
+    return 0;
+  }
+  BT_PDL_OK("rmsnorm_add", launch_pdl(rmsnorm_add_kernel<TOut>, grid, block, 0, stream, 1, p));
+  return 0;
 }
 
 // out[r] = a N(z) + b N(z^2) + c N(z^3) + e over a row z = x[r], powers element by element, N(v) = v / sqrt(mean(v^2) + eps);
@@ -447,20 +585,19 @@ extern "C" int bt_token_shift(const float* x, const float* shift, float* state, 
   return 0;
 }
 
-extern "C" int bt_rmsnorm_add(const float* x, const float* weight, float* stream_rows, const float* next_weight,
-                              void* next_out, int next_dtype, long long n_rows, int width, float eps, float factor,
-                              cudaStream_t stream) {
+extern "C" int bt_rmsnorm_add(const float* x, const int* place, int top, const float* extra, const float* weight,
+                              float* stream_rows, const float* next_weight, void* next_out, int next_dtype,
+                              long long n_rows, int width, float eps, float factor, cudaStream_t stream) {
   using namespace bt;
   BT_CHECK(n_rows >= 0 && n_rows < (1ll << 31) && width > 0, "rmsnorm_add: bad sizes rows=%lld width=%d", n_rows, width);
+  BT_CHECK(place == nullptr || top > 0, "rmsnorm_add: %d gathered rows a row", top);
   BT_CHECK(next_out == nullptr || next_dtype == kF32 || next_dtype == kBF16, "rmsnorm_add: the next rows need a known dtype");
   if (n_rows == 0) return 0;
-  if (next_out != nullptr && next_dtype == kBF16)
-    BT_PDL_OK("rmsnorm_add", launch_pdl(rmsnorm_add_kernel<__nv_bfloat16>, dim3((unsigned)n_rows), dim3(128), 0, stream, 1, x,
-                                        weight, stream_rows, next_weight, (__nv_bfloat16*)next_out, width, eps, factor));
-  else
-    BT_PDL_OK("rmsnorm_add", launch_pdl(rmsnorm_add_kernel<float>, dim3((unsigned)n_rows), dim3(128), 0, stream, 1, x, weight,
-                                        stream_rows, next_weight, (float*)next_out, width, eps, factor));
-  return 0;
+  NormAddArgs p;
+  p.x = x; p.place = place; p.top = top; p.extra = extra; p.weight = weight; p.stream_rows = stream_rows;
+  p.next_weight = next_weight; p.next_out = next_out; p.width = width; p.eps = eps; p.factor = factor;
+  if (next_out != nullptr && next_dtype == kBF16) return launch_norm_add<__nv_bfloat16>(p, n_rows, stream);
+  return launch_norm_add<float>(p, n_rows, stream);
 }
 
 extern "C" int bt_polynorm(const void* x, const float* coef, void* out, long long n_rows, int width, float eps, int dtype,

@@ -56,7 +56,8 @@ class ModelPlan:
     # learned vectors that calls of the schedule add to the stream before they run (`LayerCall.opens`)
     stream_vectors: Part | None = None
     # tensors that live for one step and that layers hand to later layers of the same step: name -> (channels, dtype);
-    # every step gets `ctx.shared[name]`, [tokens, channels], out of its scratch memory before the first layer runs
+    # every step gets `ctx.shared[name]`, [tokens, channels], out of its scratch memory before the first layer runs (a
+    # dtype of None is the step's compute type)
     step_tensors: dict = dataclasses.field(default_factory=dict)
 
     def __post_init__(self):
@@ -109,7 +110,7 @@ class ModelPlan:
         """Runs the step's tokens through every layer call; returns 32-bit logits at the wanted rows."""
         residual = ctx.ws.take((ctx.n_tokens, self.width), torch.float32)
         self.embedding.forward(ctx, self.positions, residual)
-        ctx.shared = {name: ctx.ws.take((ctx.n_tokens, channels), dtype)
+        ctx.shared = {name: ctx.ws.take((ctx.n_tokens, channels), dtype or ctx.dtype)
                       for name, (channels, dtype) in self.step_tensors.items()}
         for index, call in enumerate(self.schedule):
             entry, owns = self.cache_entry(index)

@@ -1164,15 +1164,24 @@ def latent_decode_finish(uv_heads, out, *, n_tokens, n_splits, scratch=None, mix
 
 # ---- a sublayer's normed result into the stream; the polynomial activation; the half-split rotation -----------------
 
-def rmsnorm_add(x, weight, stream_rows, eps: float, *, n_rows, next_weight=None, next_out=None, factor: float = 1.0):
-    """stream_rows[r] += factor * x[r] / sqrt(mean(x[r]^2) + eps) * weight for contiguous 32-bit [rows, width] tensors.
-    With `next_out` ([rows, width], 32-bit or bfloat16) the updated row is also written there: normed again with
-    `next_weight`, or, without one, as it is (rounded to next_out's type)."""
+def rmsnorm_add(x, weight, stream_rows, eps: float, *, n_rows, next_weight=None, next_out=None, factor: float = 1.0,
+                place=None, top: int = 0, extra=None):
+    """stream_rows[r] += factor * v[r] / sqrt(mean(v[r]^2) + eps) * weight for contiguous 32-bit [rows, width] tensors, v = x.
+    With `place` (int32) v[r] is the sum of the `top` rows x[place[r * top + j]] in that order (routed experts' results,
+    weighted, as `moe_expert` leaves them); `extra` [rows, width] is added to v.  With `next_out` ([rows, width], 32-bit or
+    bfloat16) the updated row is also written there: normed again with `next_weight`, or, without one, as it is (rounded
+    to next_out's type)."""
     width = weight.shape[0]
     _need(x, "x", torch.float32, (None, width))
     _need(stream_rows, "stream_rows", torch.float32, (None, width))
     _need(weight, "weight", torch.float32, (width,))
-    if min(x.shape[0], stream_rows.shape[0]) < n_rows:
+    if place is not None:
+        _need(place, "place", torch.int32)
+        if top <= 0 or place.numel() < n_rows * top or x.shape[0] < n_rows * top:
+            raise ShapeError(f"rmsnorm_add: {n_rows} rows of {top} gathered rows each asked of shorter tensors")
+    if extra is not None:
+        _need(extra, "extra", torch.float32, (None, width))
+    if min(x.shape[0], stream_rows.shape[0], n_rows if extra is None else extra.shape[0]) < n_rows:
         raise ShapeError(f"rmsnorm_add: {n_rows} rows asked of shorter tensors")
     if next_weight is not None and next_out is None:
         raise ShapeError("rmsnorm_add: the second norm needs a place for its rows")
@@ -1182,8 +1191,10 @@ def rmsnorm_add(x, weight, stream_rows, eps: float, *, n_rows, next_weight=None,
         _need(next_out, "next_out", (torch.float32, torch.bfloat16), (None, width))
         if next_out.shape[0] < n_rows:
             raise ShapeError(f"rmsnorm_add: {n_rows} rows asked of next_out[{next_out.shape[0]}]")
-    _work(0.0, n_rows * width * (12.0 + (next_out.element_size() if next_out is not None else 0)))
-    _check(library().bt_rmsnorm_add(_ptr(x), _ptr(weight), _ptr(stream_rows), _ptr(next_weight), _ptr(next_out),
+    _work(0.0, n_rows * width * (8.0 + 4.0 * (top if place is not None else 1) + (4.0 if extra is not None else 0.0)
+                                 + (next_out.element_size() if next_out is not None else 0)))
+    _check(library().bt_rmsnorm_add(_ptr(x), _ptr(place), c_int(top), _ptr(extra), _ptr(weight), _ptr(stream_rows),
+                                    _ptr(next_weight), _ptr(next_out),
                                     c_int(_code(next_out.dtype)) if next_out is not None else c_int(0),
                                     c_longlong(n_rows), c_int(width), c_float(eps), c_float(factor), _stream()))
 

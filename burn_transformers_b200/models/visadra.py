@@ -19,6 +19,8 @@ from ..parts import (GatedFeedForward, InterleavedRotary, LatentAttention, Linea
                      OutputNormBlock, RmsNorm, RoutedFeedForward, TokenEmbedding)
 from ..weights.spec import Concat, Stored
 
+ROUNDED_STREAM = "rounded_stream"      # the step tensor in which a layer hands the stream, rounded, to the next layer
+
 
 def _norm(names, name, width, eps):
     norm = RmsNorm(width, eps, one_gain=True)
@@ -92,13 +94,14 @@ def build_visadra(config: VisadraConfig) -> ModelPlan:
             feed_forward = (_gated(names, sources, p + "mlp.", width, mlp["ff"], std) if mlp["kind"] == "dense"
                             else _routed(names, sources, p + "mlp.", width, mlp, std))
             norm2 = _norm(names, p + "norm2", width, eps)
-        blocks.append(OutputNormBlock(mixer, norm1, feed_forward, norm2))
+        blocks.append(OutputNormBlock(mixer, norm1, feed_forward, norm2, rows=ROUNDED_STREAM, first=i == 0,
+                                      last=i == len(config.layers) - 1))
     # (a layer without a feed-forward has no use for a second norm; a file may hold its number all the same)
     ignored = frozenset(f"l{i}.norm2" for i, layer in enumerate(config.layers) if layer.get("mlp") is None)
     return ModelPlan(config=config, embedding=embedding, positions=NoPositions(), blocks=blocks,
                      schedule=[LayerCall(i) for i in range(len(blocks))], final_norm=final_norm, readout=readout,
                      names=names, vocab=config.vocab, width=width, max_context=UNBOUNDED_CONTEXT, sources=sources,
-                     ignored=ignored)
+                     ignored=ignored, step_tensors={ROUNDED_STREAM: (width, None)})
 
 
 VISADRA = register_architecture(Architecture("visadra", VisadraConfig.MODEL_TYPES, VisadraConfig, build_visadra),

@@ -211,18 +211,27 @@ class OutputNormBlock(Block):
     `shift` (parts.token_shift.TokenShift) the mixer reads every row blended with the row of the token before it.
 
     A sublayer leaves its result in a 32-bit buffer (zeroed first for parts that can only add); one kernel
-    (csrc/rowwise.cu: rmsnorm_add) norms the buffer, adds m times the result to the stream and, where the feed-forward
-    follows, writes the new row in the products' type for it in the same pass.  Both norms are RMS norms of one eps."""
+    (csrc/rowwise.cu: rmsnorm_add) norms the buffer, adds m times the result to the stream and, where another sublayer
+    follows, writes the new row in the products' type for it in the same pass.  Routed experts leave their rows unsummed
+    (`forward_pairs`): the same kernel gathers a token's rows, adds the shared expert's, and norms the sum.  Both norms are
+    RMS norms of one eps.
+
+    `rows` names a step tensor (ModelPlan.step_tensors: the stream's width, compute type) in which the layers of a model
+    hand the rounded stream from one to the next; `first` marks the layer that fills it, `last` the one after which nobody
+    reads it.  Without it a layer rounds the stream for itself."""
 
     def __init__(self, mixer: Mixer, norm1: Norm, feed_forward: FeedForward | None = None, norm2: Norm | None = None,
-                 *, scale: float = 1.0, shift=None):
+                 *, scale: float = 1.0, shift=None, rows: str | None = None, first: bool = True, last: bool = True):
         if (norm2 is None) != (feed_forward is None):
             raise ValueError("a block has both a feed-forward and the norm of its output, or neither")
         norms = [n for n in (norm1, norm2) if n is not None]
         if any(getattr(n, "has_bias", True) or n.eps != norm1.eps or not hasattr(n, "offset") for n in norms):
             raise ValueError("the norms of the sublayers' outputs are RMS norms with one eps")
+        if rows is not None and shift is not None:
+            raise ValueError("a layer with a token shift reads the 32-bit stream, not the rounded rows of the layer before")
         self.mixer, self.norm1, self.feed_forward, self.norm2 = mixer, norm1, feed_forward, norm2
         self.scale, self.shift = float(scale), shift
+        self.rows, self.first, self.last = rows, first or rows is None, last or rows is None
 
     def parts(self):
         found = {"mixer": self.mixer, "norm1": self.norm1}
@@ -253,14 +262,17 @@ class OutputNormBlock(Block):
         exact = ctx.dtype == torch.float32
         mark = ctx.ws.mark()
         branch = ctx.ws.take((n, width), torch.float32)
-        rows = ctx.ws.take((n, width), ctx.dtype) if (self.shift is not None or not exact) else None
+        rows = None
+        if self.shift is not None or not exact:
+            rows = ctx.shared[self.rows] if self.rows is not None else ctx.ws.take((n, width), ctx.dtype)
         if self.shift is not None:
             self.shift.forward(ctx, residual, rows, entry)
             x = rows
         elif exact:
             x = residual
         else:
-            rows[:n].copy_(residual[:n])
+            if self.first:
+                rows[:n].copy_(residual[:n])
             x = rows
         inner = ctx.ws.mark()
         # (a part that can store its result instead of adding it needs no zeroed buffer: one launch less a sublayer)
@@ -270,19 +282,58 @@ class OutputNormBlock(Block):
             branch.zero_()
             self.mixer.forward(ctx, x, branch, entry, owns_cache)
         ctx.ws.release(inner)
+        handed_on = None if exact or self.last else rows
         if self.feed_forward is None:
-            kernels.rmsnorm_add(branch, self.norm1.t_weight, residual, self.norm1.eps, n_rows=n, factor=self.scale)
+            kernels.rmsnorm_add(branch, self.norm1.t_weight, residual, self.norm1.eps, n_rows=n, factor=self.scale,
+                                next_out=handed_on)
             ctx.ws.release(mark)
             return
         # the feed-forward reads the new rows of the stream: as they are in 32-bit, else rounded by the same kernel
         kernels.rmsnorm_add(branch, self.norm1.t_weight, residual, self.norm1.eps, n_rows=n, factor=self.scale,
                             next_out=None if exact else rows)
         x = residual if exact else rows
+        if getattr(self.feed_forward, "sums_pairs_later", False):
+            part, place, shared = self._experts(ctx, x, branch)
+            kernels.rmsnorm_add(part, self.norm2.t_weight, residual, self.norm2.eps, n_rows=n, factor=self.scale,
+                                place=place, top=self.feed_forward.top, extra=shared, next_out=handed_on)
+            ctx.ws.release(mark)
+            return
         more = {"x32": residual} if getattr(self.feed_forward, "wants_x32", False) else {}
         if getattr(self.feed_forward, "can_store", False):
             self.feed_forward.forward(ctx, x, branch, store=True, **more)
         else:
             branch.zero_()
             self.feed_forward.forward(ctx, x, branch, **more)
-        kernels.rmsnorm_add(branch, self.norm2.t_weight, residual, self.norm2.eps, n_rows=n, factor=self.scale)
+        kernels.rmsnorm_add(branch, self.norm2.t_weight, residual, self.norm2.eps, n_rows=n, factor=self.scale,
+                            next_out=handed_on)
         ctx.ws.release(mark)
+
+    def _experts(self, ctx, x, branch):
+        """(rows of the routed experts, places, the shared expert's rows or None).  The shared expert needs nothing of the
+        routed ones: in steps of up to ParallelBlock.side_by_side_up_to tokens it runs beside them on a stream of its own."""
+        ff = self.feed_forward
+        if ff.shared is None:
+            return (*ff.forward_pairs(ctx, x), None)
+        if ctx.n_tokens > ParallelBlock.side_by_side_up_to or branch.device.type != "cuda":
+            self._run_shared(ctx, x, branch)
+            return (*ff.forward_pairs(ctx, x), branch)
+        side, = ParallelBlock._sides(branch.device, 1)
+        held, ctx.ws.hold = ctx.ws.hold, True
+        step_side, ctx.side = getattr(ctx, "side", None), None
+        try:
+            side.fork()
+            with side.stream_context():
+                self._run_shared(ctx, x, branch)
+            part, place = ff.forward_pairs(ctx, x)
+        finally:
+            side.join()
+            ctx.ws.hold, ctx.side = held, step_side
+        return part, place, branch
+
+    def _run_shared(self, ctx, x, branch):
+        shared = self.feed_forward.shared
+        if getattr(shared, "can_store", False):
+            shared.forward(ctx, x, branch, store=True)
+        else:
+            branch.zero_()
+            shared.forward(ctx, x, branch)

@@ -110,17 +110,37 @@ class RoutedFeedForward(FeedForward):
 
     def forward_routed(self, ctx, x, residual, x32=None, store=False):
         """The routed experts alone (the shared one is a feed-forward of its own and may run beside them)."""
-        if getattr(ctx, "program", None) is not None:
-            from ..engine.program import ProgramUnsupported
-            raise ProgramUnsupported("routed experts have no phase in the fused step")
-        n, top, e = ctx.n_tokens, self.top, self.n_experts
-        routes = e + self.identity
         if self.identity and x32 is None:
             if x.dtype != torch.float32:
                 raise ShapeError("routed feed-forward: experts that hand their input on need the 32-bit rows (x32)")
             x32 = x
-        pairs = n * top
         mark = ctx.ws.mark()
+        part, place, ids, weights = self._pairs(ctx, x)
+        if self.identity:
+            kernels.moe_combine(part, place, residual, n_tokens=ctx.n_tokens, top=self.top, ids=ids, weights=weights,
+                                identity_input=x32, n_stored=self.n_experts, store=store)
+        else:
+            kernels.moe_combine(part, place, residual, n_tokens=ctx.n_tokens, top=self.top, store=store)
+        ctx.ws.release(mark)
+
+    @property
+    def sums_pairs_later(self) -> bool:
+        """Whether `forward_pairs` says all there is about the routed experts' result."""
+        return self.identity == 0
+
+    def forward_pairs(self, ctx, x):
+        """The routed experts' results without the sum over a token's choices, for a consumer that sums them itself: (rows
+        sorted by expert, 32-bit and weighted [tokens * top, width]; the row of every (token, choice) pair).  Both lie in
+        the step's scratch: the caller takes a mark before and releases it when they are read."""
+        part, place, _, _ = self._pairs(ctx, x)
+        return part, place
+
+    def _pairs(self, ctx, x):
+        if getattr(ctx, "program", None) is not None:
+            from ..engine.program import ProgramUnsupported
+            raise ProgramUnsupported("routed experts have no phase in the fused step")
+        n, top, routes = ctx.n_tokens, self.top, self.n_experts + self.identity
+        pairs = n * top
         ids = ctx.ws.take((n, top), torch.int32)
         weights = ctx.ws.take((n, top), torch.float32)
         kernels.moe_route(x, self.t_router_weight, ids, weights, n_tokens=n, top=top, n_groups=self.n_groups,
@@ -138,9 +158,4 @@ class RoutedFeedForward(FeedForward):
                            activation=self.activation, limit=self.limit, gated=self.gated)
         part = ctx.ws.take((pairs, self.width), torch.float32)
         kernels.moe_expert(False, hidden, self.w_out, part, offsets, tile_first, order, weights, pairs=pairs, top=top)
-        if self.identity:
-            kernels.moe_combine(part, place, residual, n_tokens=n, top=top, ids=ids, weights=weights, identity_input=x32,
-                                n_stored=e, store=store)
-        else:
-            kernels.moe_combine(part, place, residual, n_tokens=n, top=top, store=store)
-        ctx.ws.release(mark)
+        return part, place, ids, weights

@@ -50,12 +50,12 @@ def average_case(rng, width, news, dtype, shift=0.0):
 @pytest.mark.parametrize("width", [1, 7, 64, 70, 130, 1104])
 def test_gated_average_of_unequal_runs_with_a_state_carried_over(dtype, tol, width):
     """Several steps on the same slots: single tokens, short runs, runs at and beside what a warp (8 tokens), a block
-    (128) and a cluster (up to 1,024) hold, and one that goes round the cluster's loop; slots that no sequence names
+    (64) and a cluster (up to 512) hold, and some that go round the cluster's loop; slots that no sequence names
     keep their state, rows behind the step's stay as they are."""
     rng = np.random.default_rng(width)
     state = dev(rng.standard_normal((9, width)))
     for news, slots in (([1], [4]), ([1, 1, 1, 1, 1], [3, 0, 6, 1, 8]), ([2, 16, 1, 9], [5, 2, 0, 3]), ([17, 1, 8, 128], [1, 7, 4, 0]),
-                        ([129, 127, 3], [2, 6, 5]), ([1023, 1, 1025], [0, 1, 2]), ([130, 2300], [8, 3])):
+                        ([129, 63, 3], [2, 6, 5]), ([65, 64, 24], [6, 5, 7]), ([513, 1, 512, 1025], [0, 1, 2, 6]), ([130, 2300], [8, 3])):
         proj, zb, xb, z, values, gate = average_case(rng, width, news, dtype)
         before = host(state).clone()
         n = sum(news)
@@ -255,3 +255,34 @@ def test_attention_of_fresh_prompts_with_a_sink_and_no_gate(heads, dq, dv):
             want = plain.softmax_beside_a_sink(scores, seen, host(sink)[h]) @ host(v[at:at + count, h])
             assert np.abs(np.asarray(host(out[at:at + count, h]) - want)).max() < 2e-2 * max(0.3, float(want.abs().max()))
         at += count
+
+
+@pytest.mark.parametrize("width", [70, 64, 516, 1000, 2000, 3000, 4096, 4100, 5000])
+@pytest.mark.parametrize("top, extra", [(0, False), (0, True), (3, False), (1, True), (6, True)])
+def test_norm_added_over_gathered_rows(width, top, extra):
+    """A token's rows gathered by place and summed with the shared expert's, normed, added to the stream, and handed on
+    as they are, normed, or not at all; rows behind the last stay as they are."""
+    rng = np.random.default_rng(width + top)
+    n, eps = 9, 1e-3
+    rows = n * max(1, top)
+    x, stream = dev(rng.standard_normal((rows, width))), dev(rng.standard_normal((n + 1, width)))
+    weight, after = dev(rng.standard_normal(width)), dev(rng.standard_normal(width))
+    more = dev(rng.standard_normal((n, width))) if extra else None
+    order = rng.permutation(rows)
+    before = host(stream).clone()
+    value = host(x)[torch.tensor(order)].view(n, -1, width).sum(1) if top else host(x)
+    if extra:
+        value = value + host(more)
+    want = before[:n] + 0.7 * plain.rms_divide(value, eps) * host(weight)
+    gathered = dict(place=ints(order), top=top) if top else {}
+    for next_weight, next_dtype in ((None, None), (None, torch.bfloat16), (after, torch.float32), (after, torch.bfloat16)):
+        stream.copy_(before)
+        out = None if next_dtype is None else torch.full((n + 1, width), 9.0, dtype=next_dtype, device=DEV)
+        kernels.rmsnorm_add(x, weight, stream, eps, n_rows=n, factor=0.7, extra=more, next_weight=next_weight, next_out=out,
+                            **gathered)
+        assert rel(host(stream[:n]), want) < 1e-5 and torch.equal(host(stream[n]), before[n])
+        if out is None:
+            continue
+        handed = want if next_weight is None else plain.rms_divide(want, eps) * host(after)
+        assert rel(host(out[:n]), handed) < (1e-5 if next_dtype == torch.float32 else 1e-2)
+        assert bool((out[n] == 9.0).all())
