@@ -104,6 +104,11 @@ int bt_sink_attention(const void* q, long long q_row, int q_head, const void* k,
                       void* out, long long out_row, int out_head, const int* seq_start, const float* sink, int n_seqs,
                       int max_new, int n_heads, int dq, int dv, float scale, int window, int keep_first, int kv_group,
                       int sigmoid, const float* bias, cudaStream_t stream);
+int bt_sink_attention_tcgen05_supports(int dq, int dv, long long q_row, long long gate_row, int gate_head);
+int bt_sink_attention_tcgen05(const void* q, long long q_row, const void* k, const void* v, long long rows, const void* gate,
+                              long long gate_row, int gate_head, void* out, int* status, const int* seq_start,
+                              const int* past_len, const float* sink, int n_seqs, int max_new, int n_heads, int dq, int dv,
+                              float scale, int window, cudaStream_t stream);
 int bt_head_linear(const void* a, long long a_row_stride, int a_head_stride, const void* w, void* out,
                    long long out_row_stride, int out_head_stride, const void* gate, long long gate_row_stride,
                    int gate_head_stride, int n_tokens, int n_heads, int K, int N, int tensor_cores, int dtype,

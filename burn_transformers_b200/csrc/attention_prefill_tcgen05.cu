@@ -30,6 +30,12 @@
 // bias[head]) and nothing is normalised, so the two threads of a row exchange no maximum, nothing is rescaled and
 // nothing divided at the end.  With a window, positions below `keep_first` stay visible to every later query: the tiles
 // that hold them and lie before the window's first tile are walked first (the products never ask where a tile lies).
+//
+// The softmax form also takes heads whose channels are fewer than HD and HV (any multiples of 8): keys and values then
+// lie head by head, [head][token][channels], so that a box that reaches past a head's channels is filled with zeros by
+// the TMA; the queries' boxes may reach into the next head's channels, which meet those zeros.  Output channels past a
+// value head's are not stored.  A sink, a number per head, adds exp(sink) to the softmax's denominator; a gate multiplies
+// the result by sigmoid(gate).
 #include "api.h"
 #include "common.cuh"
 #include "tma.cuh"
@@ -56,6 +62,13 @@ struct TaParams {
   int causal, window;
   int keep_first;              // SIGMOID, with a window: positions below this stay visible
   const float* bias;           // SIGMOID: a number per head added to the scaled score (may be null)
+  int q_head_cols;             // columns between query heads in a row of the projections
+  int v_dim;                   // channels of a value head (at most HV), which lie side by side in `out`
+  int kv_rows;                 // > 0: keys and values lie head by head, this many rows each (row: a token of the step)
+  const float* sink;           // softmax: a number per head whose exponential joins the denominator (may be null)
+  const __nv_bfloat16* gate;   // multiplies the result by sigmoid(gate) (may be null)
+  long long gate_row;          // elements between tokens and between heads of the gate
+  int gate_head;
 };
 
 __device__ __forceinline__ unsigned ta_smem(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -253,7 +266,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
       ta_bar_expect(q_full, TILE_BYTES);
       for (int cb = 0; cb < CB; ++cb)
         for (int h = 0; h < 2; ++h)
-          ta_tma(Qs + cb * 2 * TA_BOX_BYTES + h * TA_BOX_BYTES, &q_map, head * HD + cb * 64, t0 + q0 + h * 64, q_full);
+          ta_tma(Qs + cb * 2 * TA_BOX_BYTES + h * TA_BOX_BYTES, &q_map, head * p.q_head_cols + cb * 64, t0 + q0 + h * 64, q_full);
       // where the 64 keys of half h of tile `it` lie: their row in the tensor and the first columns of K and V
       auto where = [&](int it, int h, int& row, int& col_k, int& col_v) {
         const int kt = tile_at(it);
@@ -262,6 +275,9 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
           const int key = min(kt * TA_BK + h * 64, kv_len - 1);
           const int page = p.table[(long long)seq * p.table_stride + (key / 64) % p.table_len];
           row = (page * p.n_kv_heads + kv_head) * 64;
+          col_k = col_v = 0;
+        } else if (p.kv_rows > 0) {
+          row = kv_head * p.kv_rows + t0 + kt * TA_BK + h * 64;
           col_k = col_v = 0;
         } else {
           row = t0 + kt * TA_BK + h * 64;
@@ -530,10 +546,30 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
     }
     if (!ok) *failed = 1;
     if (ok && r < nq) {
-      const float inv = SIGMOID ? 1.f : (l > 0.f ? 1.f / l : 0.f);
-      __nv_bfloat16* dst = p.out + (long long)(t0 + q0 + r) * ((long long)p.n_heads * HV) + head * HV + half * HH;
+      float inv = SIGMOID ? 1.f : (l > 0.f ? 1.f / l : 0.f);
+      if constexpr (!SIGMOID) {
+        if (p.sink != nullptr) {       // the denominator's other term, over the larger of the two exponents
+          const float sink2 = p.sink[head] * 1.4426950408889634f, top = fmaxf(m, sink2);
+          const float mine = ta_exp2(m - top);
+          inv = mine / fmaf(l, mine, ta_exp2(sink2 - top));
+        }
+      }
+      const long long token = t0 + q0 + r;
+      __nv_bfloat16* dst = p.out + token * ((long long)p.n_heads * p.v_dim) + head * p.v_dim + half * HH;
+      const __nv_bfloat16* gate = p.gate != nullptr ? p.gate + token * p.gate_row + (long long)head * p.gate_head + half * HH : nullptr;
 #pragma unroll
       for (int c = 0; c < HH; c += 8) {
+        if (half * HH + c >= p.v_dim) continue;
+        if (gate != nullptr) {
+          const uint4 raw = *reinterpret_cast<const uint4*>(gate + c);
+          const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const float2 g = __bfloat1622float2(g2[i]);
+            o[c + 2 * i] *= __fdividef(1.f, 1.f + __expf(-g.x));
+            o[c + 2 * i + 1] *= __fdividef(1.f, 1.f + __expf(-g.y));
+          }
+        }
         uint4 x;
         x.x = ta_pack(o[c] * inv, o[c + 1] * inv);
         x.y = ta_pack(o[c + 2] * inv, o[c + 3] * inv);
@@ -619,7 +655,8 @@ static int run_attention_prefill_tcgen05(const void* q, long long q_rows, long l
     if (int rc = tensor_map_2d_bf16(&vm, v, rows, v_dim, row_stride, 64)) return rc;
   }
   TaParams p{(__nv_bfloat16*)out, seq_start, past_len, kv_table, table_stride, table_len > 0 ? table_len : 1, status,
-             n_heads, n_kv_heads, k_col, v_col, scale * 1.4426950408889634f, causal, window, keep_first, bias};
+             n_heads, n_kv_heads, k_col, v_col, scale * 1.4426950408889634f, causal, window, keep_first, bias,
+             head_dim, v_dim, 0, nullptr, nullptr, 0, 0};
   BT_CHECK((v_dim == 64 || v_dim == 128) && (sigmoid || v_dim == head_dim),
            "attention_prefill_tcgen05: values of %d channels beside keys of %d are not supported", v_dim, head_dim);
   if (sigmoid) {
@@ -657,4 +694,40 @@ extern "C" int bt_sigmoid_attention_tcgen05(const void* q, long long q_rows, lon
   return run_attention_prefill_tcgen05(q, q_rows, q_row_stride, k, v, pool_pages, kv_table, table_stride, table_len, page_size,
                                        out, status, seq_start, past_len, n_seqs, max_new, n_heads, n_kv_heads, head_dim, scale,
                                        1, window, 1, bias, keep_first, pool_row_stride, v_dim, stream);
+}
+
+// Causal multi-head attention of sequences that start at position 0 with a sink and an output gate (each optional): query
+// head h at columns h * dq of the rows of `q`; keys [n_heads][rows][dq] and values [n_heads][rows][dv], rows: the step's
+// tokens; dq and dv multiples of 8, at most 128.  out: [tokens, n_heads * dv].
+extern "C" int bt_sink_attention_tcgen05_supports(int dq, int dv, long long q_row, long long gate_row, int gate_head) {
+  return dq > 0 && dv > 0 && dq <= 128 && dv <= 128 && dq % 8 == 0 && dv % 8 == 0 && q_row % 8 == 0 && gate_row % 8 == 0 &&
+         gate_head % 8 == 0;
+}
+
+extern "C" int bt_sink_attention_tcgen05(const void* q, long long q_row, const void* k, const void* v, long long rows,
+                                         const void* gate, long long gate_row, int gate_head, void* out, int* status,
+                                         const int* seq_start, const int* past_len, const float* sink, int n_seqs,
+                                         int max_new, int n_heads, int dq, int dv, float scale, int window,
+                                         cudaStream_t stream) {
+  using namespace bt;
+  BT_CHECK(bt_sink_attention_tcgen05_supports(dq, dv, q_row, gate_row, gate_head),
+           "sink_attention_tcgen05: sizes or strides the kernel does not take (dq=%d dv=%d)", dq, dv);
+  auto at16 = [](const void* ptr) { return (unsigned long long)ptr % 16 == 0; };
+  BT_CHECK(at16(q) && at16(k) && at16(v) && at16(out) && at16(gate), "sink_attention_tcgen05: operands must lie on 16-byte boundaries");
+  BT_CHECK(n_heads > 0 && n_heads <= 65535 && n_seqs <= 65535 && window >= 0 && rows >= 1 && rows * n_heads < (1ll << 31) &&
+               (long long)n_heads * dq <= q_row,
+           "sink_attention_tcgen05: bad sizes heads=%d sequences=%d rows=%lld", n_heads, n_seqs, rows);
+  if (n_seqs == 0 || max_new == 0) return 0;
+  CUtensorMap qm, km, vm;
+  if (int rc = tensor_map_2d_bf16(&qm, q, (unsigned long long)rows, (unsigned long long)n_heads * dq, (unsigned long long)q_row, 64))
+    return rc;
+  if (int rc = tensor_map_2d_bf16(&km, k, (unsigned long long)rows * n_heads, dq, dq, 64)) return rc;
+  if (int rc = tensor_map_2d_bf16(&vm, v, (unsigned long long)rows * n_heads, dv, dv, 64)) return rc;
+  TaParams p{(__nv_bfloat16*)out, seq_start, past_len, nullptr, 0, 1, status, n_heads, n_heads, 0, 0,
+             scale * 1.4426950408889634f, 1, window, 0, nullptr, dq, dv, (int)rows, sink, (const __nv_bfloat16*)gate,
+             gate_row, gate_head};
+  if (dq <= 64 && dv <= 64) return launch_ta<64, 64, false>(qm, km, vm, p, n_seqs, max_new, stream);
+  if (dq <= 64) return launch_ta<64, 128, false>(qm, km, vm, p, n_seqs, max_new, stream);
+  if (dv <= 64) return launch_ta<128, 64, false>(qm, km, vm, p, n_seqs, max_new, stream);
+  return launch_ta<128, 128, false>(qm, km, vm, p, n_seqs, max_new, stream);
 }

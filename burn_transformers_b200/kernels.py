@@ -1081,20 +1081,49 @@ def sink_attention_supports(q, k, v, gate, out) -> bool:
                                                      c_int(gh), c_longlong(orow), c_int(oh)))
 
 
-def sink_attention(q, k, v, out, seq_start, *, n_seqs, max_new, scale, sink=None, gate=None, window=0):
+def sink_attention_tcgen05_supports(q, k, v, gate, out) -> bool:
+    """Whether the tcgen05 form takes these views: bfloat16, heads of up to 128 channels in multiples of 8, query heads side
+    by side in a row, keys and values head by head ([heads, tokens, channels] in memory), out contiguous."""
+    if any(t is not None and t.dtype is not torch.bfloat16 for t in (q, k, v, gate, out)):
+        return False
+    (qr, qh), (kr, kh), (vr, vh), (gr, gh), (orow, oh) = _sink_attention_strides(q, k, v, gate, out)
+    n, heads, dq, dv = q.shape[0], q.shape[1], q.shape[2], v.shape[2]
+    if k.shape[0] != n or v.shape[0] != n or (qh, kr, kh, vr, vh, orow, oh) != (dq, dq, n * dq, dv, n * dv, heads * dv, dv):
+        return False
+    if any(t is not None and t.data_ptr() % 16 for t in (q, k, v, gate, out)):
+        return False
+    return _supports("bt_sink_attention_tcgen05_supports", dq, dv, qr, gr, gh)
+
+
+def sink_attention(q, k, v, out, seq_start, *, n_seqs, max_new, scale, sink=None, gate=None, window=0, past_len=None, impl=None):
     """Causal multi-head attention of sequences that start at position 0, on tensor cores (bfloat16): token t of a
     sequence sees the sequence's tokens up to itself.  q, k: views [tokens, heads, dq]; v, out, gate: views
     [tokens, heads, dv].  `sink` [heads] adds exp(sink_h) to head h's softmax denominator; `gate` multiplies the result by
-    sigmoid(gate).  Scores, softmax and sums are 32-bit."""
+    sigmoid(gate).  Scores, softmax and sums are 32-bit.  With `past_len` (int32, zeros: one a sequence) and views that
+    sink_attention_tcgen05_supports takes, both products are tcgen05.mma with the scores in tensor memory
+    (csrc/attention_prefill_tcgen05.cu), else mma.sync (csrc/sink_attention_mma.cu); `impl` ("tcgen05", "mma") asks for one
+    by name."""
     heads, dq, dv = q.shape[1], q.shape[2], v.shape[2]
-    if not sink_attention_supports(q, k, v, gate, out):
+    if impl is None:
+        impl = "tcgen05" if past_len is not None and sink_attention_tcgen05_supports(q, k, v, gate, out) else "mma"
+    supports = sink_attention_tcgen05_supports if impl == "tcgen05" else sink_attention_supports
+    if not supports(q, k, v, gate, out):
         raise ShapeError("sink_attention: the kernel does not take these views (see sink_attention_supports)")
     if sink is not None:
         _need(sink, "sink", torch.float32, (heads,))
     (qr, qh), (kr, kh), (vr, vh), (gr, gh), (orow, oh) = _sink_attention_strides(q, k, v, gate, out)
     if _PROFILE is not None:
         ctx = float(_PROFILE.context_hint or 0)
-        _work(2.0 * q.shape[0] * heads * (ctx / 2) * (dq + dv), 2.0 * q.shape[0] * heads * (2 * dq + 2 * dv))
+        seen = ctx / 2 if not window or window >= ctx else window - window * window / (2.0 * ctx)
+        _work(2.0 * q.shape[0] * heads * seen * (dq + dv), 2.0 * q.shape[0] * heads * (2 * dq + 2 * dv))
+    if impl == "tcgen05":
+        _need(past_len, "past_len", torch.int32)
+        _check(library().bt_sink_attention_tcgen05(_ptr(q), c_longlong(qr), _ptr(k), _ptr(v), c_longlong(q.shape[0]), _ptr(gate),
+                                                   c_longlong(gr), c_int(gh), _ptr(out), _ptr(kernel_status(q.device)),
+                                                   _ptr(seq_start), _ptr(past_len), _ptr(sink), c_int(n_seqs), c_int(max_new),
+                                                   c_int(heads), c_int(dq), c_int(dv), c_float(scale), c_int(window),
+                                                   _stream()))
+        return
     _check(library().bt_sink_attention(_ptr(q), c_longlong(qr), c_int(qh), _ptr(k), c_longlong(kr), c_int(kh), _ptr(v),
                                        c_longlong(vr), c_int(vh), _ptr(gate), c_longlong(gr), c_int(gh), _ptr(out),
                                        c_longlong(orow), c_int(oh), _ptr(seq_start), _ptr(sink), c_int(n_seqs),

@@ -183,8 +183,9 @@ class LatentAttention(Mixer):
         if dtype == torch.bfloat16 and ctx.fresh and not ctx.is_decode and ctx.max_new >= self.plain_from:
             # fresh prompts: the step's own latent rows, keys and values per head, ordinary attention
             rows = ctx.ws.take((n, dk), dtype)
-            keys = ctx.ws.take((n, heads, self.dim + rot), dtype)
-            values = ctx.ws.take((n, heads, self.vdim), dtype)
+            # (head by head: the tcgen05 attention's boxes then end with a head's channels, whatever their number)
+            keys = ctx.ws.take((heads, n, self.dim + rot), dtype).transpose(0, 1)
+            values = ctx.ws.take((heads, n, self.vdim), dtype).transpose(0, 1)
             mixed = ctx.ws.take((n, self.mixed_width), dtype)
             mixed_heads = mixed.view(n, heads, self.vdim)
             if kernels.sink_attention_supports(q_heads, keys, values, gate, mixed_heads):
@@ -198,7 +199,8 @@ class LatentAttention(Mixer):
                     self.positions.rotate_vectors(ctx, q_heads[:, :, self.dim:], q_heads[:, :, self.dim:])
                 kernels.sink_attention(q_heads, keys, values, mixed_heads, ctx.seq_start, n_seqs=ctx.n_seqs,
                                        max_new=ctx.max_new, scale=self.scale,
-                                       sink=self.t_sink if self.has_sink else None, gate=gate, window=window)
+                                       sink=self.t_sink if self.has_sink else None, gate=gate, window=window,
+                                       past_len=ctx.past_len)
                 linear(ctx, mixed, self.t_out_weight, None, residual, m=n, residual=None if store else residual, w_is_nk=True)
                 ctx.ws.release(mark)
                 return

@@ -235,25 +235,45 @@ def test_latent_attention_with_a_sink(dtype, tol, tensor_cores, heads, rank, rot
             at += count
 
 
-@pytest.mark.parametrize("heads, dq, dv", [(3, 40, 24), (2, 96, 64), (4, 128, 128), (5, 72, 64), (1, 264, 16), (2, 64, 128)])
-def test_attention_of_fresh_prompts_with_a_sink_and_no_gate(heads, dq, dv):
+@pytest.mark.parametrize("impl", ["mma", "tcgen05"])
+@pytest.mark.parametrize("window, gated", [(0, False), (0, True), (70, False)])
+@pytest.mark.parametrize("heads, dq, dv", [(3, 40, 24), (2, 96, 64), (4, 128, 128), (5, 72, 56), (1, 264, 16), (2, 64, 104),
+                                           (7, 8, 8), (3, 120, 72)])
+def test_attention_of_fresh_prompts_with_a_sink(impl, window, gated, heads, dq, dv):
+    """Both kernels for prompts that start a sequence, keys and values head by head in memory: head sizes that fill the
+    tcgen05 kernel's boxes of 64 channels and that do not (what lies beyond a head must not count), several tiles of 128
+    keys, sinks that take nearly everything and nothing, a gate and a window or none."""
     rng = np.random.default_rng(dq)
-    news = [200, 1, 70, 129]
+    news = [200, 1, 70, 129, 300]
     n = sum(news)
-    q, k, v = (dev(rng.standard_normal((n, heads, d)), torch.bfloat16) for d in (dq, dq, dv))
-    out = torch.zeros((n, heads, dv), dtype=torch.bfloat16, device=DEV)
-    assert kernels.sink_attention_supports(q, k, v, None, out)
+    # (queries inside longer rows, as a projection leaves them; a large number right behind the last head's channels)
+    rows = dev(rng.standard_normal((n, heads * dq + heads * dv + 8)), torch.bfloat16)
+    rows[:, heads * (dq + dv):] = 1e4
+    q = rows[:, :heads * dq].view(n, heads, dq) if heads * dq else None
+    gate = rows[:, heads * dq:heads * (dq + dv)].view(n, heads, dv) if gated else None
+    k, v = (dev(rng.standard_normal((heads, n, d)), torch.bfloat16).transpose(0, 1) for d in (dq, dv))
+    out = torch.full((n + 1, heads, dv), 9.0, dtype=torch.bfloat16, device=DEV)
+    takes = kernels.sink_attention_tcgen05_supports(q, k, v, gate, out[:n])
+    assert takes == (dq <= 128) and kernels.sink_attention_supports(q, k, v, gate, out[:n])
+    if impl == "tcgen05" and not takes:
+        return
     sink = dev(np.linspace(-5.0, 6.0, heads) if heads > 1 else [0.7])
     scale = 1.5 / math.sqrt(dq)
-    kernels.sink_attention(q, k, v, out, ints(np.concatenate([[0], np.cumsum(news)])), n_seqs=len(news), max_new=max(news),
-                           scale=scale, sink=sink)
+    kernels.sink_attention(q, k, v, out[:n], ints(np.concatenate([[0], np.cumsum(news)])), n_seqs=len(news), max_new=max(news),
+                           scale=scale, sink=sink, gate=gate, window=window, past_len=ints([0] * len(news)), impl=impl)
+    kernels.check_status(torch.device(DEV))
+    assert bool((out[n] == 9.0).all())
     at = 0
     for count in news:
         seen = torch.ones(count, count).tril().bool()
+        if window:
+            seen &= ~torch.ones(count, count).tril(-window).bool()
         for h in range(heads):
             scores = host(q[at:at + count, h]) @ host(k[at:at + count, h]).T * scale
             want = plain.softmax_beside_a_sink(scores, seen, host(sink)[h]) @ host(v[at:at + count, h])
-            assert np.abs(np.asarray(host(out[at:at + count, h]) - want)).max() < 2e-2 * max(0.3, float(want.abs().max()))
+            if gated:
+                want = want * plain.sigmoid(host(gate[at:at + count, h]))
+            assert np.abs(np.asarray(host(out[at:at + count, h]) - want)).max() < 2e-2 * max(0.3, float(want.abs().max())), (count, h)
         at += count
 
 
