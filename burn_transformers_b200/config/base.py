@@ -116,6 +116,10 @@ class ModelConfig:
             return value
         return value
 
+    def learn_shapes(self, shapes: dict[str, tuple[int, ...]]) -> None:
+        """Takes sizes that config.json does not give from the shapes of the checkpoint's tensors (by stored name).  Called
+        between reading the configuration and building the model; most families have nothing to learn."""
+
     def validate(self) -> None:  # pragma: no cover - overridden
         raise NotImplementedError
 

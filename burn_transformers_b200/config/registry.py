@@ -10,7 +10,7 @@ import dataclasses
 from pathlib import Path
 from typing import Callable
 
-from ..errors import UnsupportedArchitecture
+from ..errors import CheckpointError, UnsupportedArchitecture
 from .base import ModelConfig, detect_model_type, read_json_object, _TEXT_WRAPPERS
 
 
@@ -62,4 +62,11 @@ def config_from_folder(folder) -> tuple[Architecture, ModelConfig]:
             if isinstance(data.get(wrapper), dict):
                 data = data[wrapper]
                 break
-    return arch, arch.config_class.from_dict(data)
+    config = arch.config_class.from_dict(data)
+    if type(config).learn_shapes is not ModelConfig.learn_shapes:
+        from ..weights.loader import discover
+        try:
+            config.learn_shapes({name: entry.shape for name, entry in discover(folder).items()})
+        except CheckpointError:
+            pass      # (no weights yet, or broken ones: loading them says what is wrong)
+    return arch, config

@@ -83,11 +83,11 @@ int bt_linear_few_tcgen05(const void* x, const void* w, const float* bias, const
 int bt_linear_stream_supports(int M, int N, int K, int fuse_ln);
 int bt_linear_stream(const void* a, const float* x32, const int* rows, const float* gamma, const float* beta, float eps,
                      const void* w, const float* bias, const float* residual, void* out, int M, int N, int K, int act,
-                     int out_is_f32, int warps_k, cudaStream_t stream);
+                     int out_is_f32, int warps_k, int rms, cudaStream_t stream);
 int bt_linear_skinny_supports(int M, int N, int K, int w_is_nk, int fuse_ln);
 int bt_linear_skinny(const void* a, const float* x32, const int* rows, const float* gamma, const float* beta, float eps,
                      const void* w, const float* bias, const float* residual, void* out, int M, int N, int K,
-                     int w_is_nk, int act, int out_is_f32, int split, cudaStream_t stream);
+                     int w_is_nk, int act, int out_is_f32, int split, int rms, cudaStream_t stream);
 // Attention over a latent cache (csrc/latent_attention.cu), the decayed linear recurrence (csrc/lightning.cu) and the
 // row-wise kernels between products (csrc/rowwise.cu).
 int bt_latent_append(const void* src, long long row_stride, const float* norm_weight, float eps, const int* positions,
@@ -98,20 +98,20 @@ int bt_latent_gather(const void* pool, const int* positions, const int* token_se
                      int table_len, int page_size, void* rows, int n_tokens, int dk, int dtype, cudaStream_t stream);
 // Causal multi-head attention of fresh prompts on tensor cores with a sink and a gate (csrc/sink_attention_mma.cu).
 int bt_sink_attention_supports(int dq, int dv, long long q_row, int q_head, long long k_row, int k_head, long long v_row,
-                               int v_head, long long gate_row, int gate_head, long long out_row, int out_head);
+                               int v_head, long long gate_row, int gate_head, int gate_step, long long out_row, int out_head);
 int bt_sink_attention(const void* q, long long q_row, int q_head, const void* k, long long k_row, int k_head,
-                      const void* v, long long v_row, int v_head, const void* gate, long long gate_row, int gate_head,
+                      const void* v, long long v_row, int v_head, const void* gate, long long gate_row, int gate_head, int gate_step,
                       void* out, long long out_row, int out_head, const int* seq_start, const float* sink, int n_seqs,
                       int max_new, int n_heads, int dq, int dv, float scale, int window, int keep_first, int kv_group,
                       int sigmoid, const float* bias, cudaStream_t stream);
-int bt_sink_attention_tcgen05_supports(int dq, int dv, long long q_row, long long gate_row, int gate_head);
+int bt_sink_attention_tcgen05_supports(int dq, int dv, long long q_row, long long gate_row, int gate_head, int gate_step);
 int bt_sink_attention_tcgen05(const void* q, long long q_row, const void* k, const void* v, long long rows, const void* gate,
-                              long long gate_row, int gate_head, void* out, int* status, const int* seq_start,
+                              long long gate_row, int gate_head, int gate_step, void* out, int* status, const int* seq_start,
                               const int* past_len, const float* sink, int n_seqs, int max_new, int n_heads, int dq, int dv,
                               float scale, int window, cudaStream_t stream);
 int bt_head_linear(const void* a, long long a_row_stride, int a_head_stride, const void* w, void* out,
                    long long out_row_stride, int out_head_stride, const void* gate, long long gate_row_stride,
-                   int gate_head_stride, int n_tokens, int n_heads, int K, int N, int tensor_cores, int dtype,
+                   int gate_head_stride, int gate_step, int n_tokens, int n_heads, int K, int N, int tensor_cores, int dtype,
                    cudaStream_t stream);
 long long bt_latent_attention_scratch_floats(int n_tokens, int n_heads, int rank, int n_splits);
 int bt_latent_attention(const void* q, long long q_row_stride, const void* pool, const int* table, int table_stride,
@@ -127,7 +127,7 @@ int bt_latent_decode_prep(const void* proj, long long row_stride, int q_off, int
                           int page_size, void* pool, void* q_latent, int n_tokens, int n_heads, int dim, int rank, int rot,
                           int owns, int dtype, cudaStream_t stream);
 int bt_latent_decode_finish(const float* part, const void* mixed_latent, int n_splits, const void* uv, const void* gate,
-                            long long gate_row_stride, void* out, long long out_row_stride, int n_tokens, int n_heads,
+                            long long gate_row_stride, int gate_per_head, void* out, long long out_row_stride, int n_tokens, int n_heads,
                             int rank, int vdim, int dtype, cudaStream_t stream);
 int bt_latent_attention_rows(int rank, int rot, int dtype, int tensor_cores);
 int bt_lightning_scan(const void* proj, long long row_stride, int q_off, int k_off, int v_off, float* state,
@@ -216,6 +216,34 @@ int bt_moe_expert(int first, const void* a, long long a_row_stride, const void* 
                   int N, int act, float limit, int tensor_cores, int dtype, cudaStream_t stream);
 int bt_moe_combine(const float* part, const int* place, float* stream_rows, long long n_tokens, int top, int width,
                    const int* ids, const float* weights, const float* input, int n_stored, int store,
+                   cudaStream_t stream);
+// Differential attention (csrc/differential_attention.cu, csrc/attention_prefill_tcgen05.cu) and gated linear attention
+// (csrc/gla.cu).
+int bt_differential_prep(const void* proj, long long row_stride, const float* conv, float* state, const int* slots,
+                         const int* seq_start, const int* token_seq, const int* positions, const float* q_weight,
+                         const float* k_weight, float eps, const float* inv_freq, int rot_dims, float rot_size, int taps,
+                         const int* table, int table_stride, int table_len, int page_size, void* pool, void* q_out, int q_pad,
+                         int n_tokens, int n_seqs, int max_new, int n_heads, int n_kv_heads, int dim, int vdim, int dtype,
+                         cudaStream_t stream);
+int bt_two_map_attention(const void* q, long long q_row_stride, int q_pad, const void* pool, const int* table, int table_stride,
+                         int table_len, int page_size, const int* token_seq, const int* positions, float* out, int n_tokens,
+                         int n_heads, int n_kv_heads, int dim, int vdim, float scale, int n_splits, int dtype,
+                         cudaStream_t stream);
+int bt_two_map_attention_tcgen05_supports(int dim, int v_dim);
+int bt_two_map_attention_tcgen05(const void* q, long long rows, int pad, const void* pool, long long pool_pages,
+                                 const int* table, int table_stride, int table_len, float* out, int* status,
+                                 const int* seq_start, const int* past_len, int n_seqs, int max_new, int n_heads,
+                                 int n_kv_heads, int dim, int v_dim, float scale, cudaStream_t stream);
+int bt_differential_combine(const float* parts, int n_splits, const float* share, float gain, float eps, void* out,
+                            long long out_row_stride, int n_tokens, int n_heads, int vdim, int dtype, cudaStream_t stream);
+int bt_gla_scan_fuses(int dim, int vdim);
+int bt_gla_scan(const void* proj, long long row_stride, int q_off, int k_off, int v_off, float q_scale, const float* dt,
+                float log_scale, float* state, const int* slots, const int* seq_start, float* out, long long out_row_stride,
+                int n_seqs, int n_heads, int dim, int vdim, const float* norm_weight, float eps, int g_off, void* mixed,
+                long long mixed_row_stride, int dtype, cudaStream_t stream);
+int bt_gla_chunked(const void* proj, long long row_stride, int q_off, int k_off, int v_off, float q_scale, const float* dt,
+                   float log_scale, float* state, const int* slots, const int* seq_start, float* out,
+                   long long out_row_stride, float* scratch, int max_new, int n_seqs, int n_heads, int dim, int vdim, int dtype,
                    cudaStream_t stream);
 int bt_add_vector(float* x, const float* vec, long long n_rows, int width, cudaStream_t stream);
 int bt_add_rows(float* x, const float* a, const float* b, const float* c, long long n, cudaStream_t stream);

@@ -34,7 +34,8 @@
 // The softmax form also takes heads whose channels are fewer than HD and HV (any multiples of 8): keys and values then
 // lie head by head, [head][token][channels], so that a box that reaches past a head's channels is filled with zeros by
 // the TMA; the queries' boxes may reach into the next head's channels, which meet those zeros.  Output channels past a
-// value head's are not stored.  A sink, a number per head, adds exp(sink) to the softmax's denominator; a gate multiplies
+// value head's are not stored.  Differential attention runs a head's two maps as two heads over one pool row [key 1 | key
+// 2 | value] (`maps`), with the queries padded by zeros to HD channels and the results left in 32-bit.  A sink, a number per head, adds exp(sink) to the softmax's denominator; a gate multiplies
 // the result by sigmoid(gate).
 #include "api.h"
 #include "common.cuh"
@@ -68,7 +69,9 @@ struct TaParams {
   const float* sink;           // softmax: a number per head whose exponential joins the denominator (may be null)
   const __nv_bfloat16* gate;   // multiplies the result by sigmoid(gate) (may be null)
   long long gate_row;          // elements between tokens and between heads of the gate
-  int gate_head;
+  int gate_head, gate_step;    // gate_step 0: one gate a head
+  float* out32;                // not null: the result as 32-bit numbers here, [tokens, n_heads * v_dim], instead of `out`
+  int maps, k_map_cols;        // paged: a pool row holds `maps` keys `k_map_cols` columns apart; head h reads key h % maps
 };
 
 __device__ __forceinline__ unsigned ta_smem(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -275,7 +278,8 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
           const int key = min(kt * TA_BK + h * 64, kv_len - 1);
           const int page = p.table[(long long)seq * p.table_stride + (key / 64) % p.table_len];
           row = (page * p.n_kv_heads + kv_head) * 64;
-          col_k = col_v = 0;
+          col_k = (head % p.maps) * p.k_map_cols;
+          col_v = 0;
         } else if (p.kv_rows > 0) {
           row = kv_head * p.kv_rows + t0 + kt * TA_BK + h * 64;
           col_k = col_v = 0;
@@ -556,11 +560,12 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
       }
       const long long token = t0 + q0 + r;
       __nv_bfloat16* dst = p.out + token * ((long long)p.n_heads * p.v_dim) + head * p.v_dim + half * HH;
-      const __nv_bfloat16* gate = p.gate != nullptr ? p.gate + token * p.gate_row + (long long)head * p.gate_head + half * HH : nullptr;
+      const __nv_bfloat16* gate = p.gate != nullptr ? p.gate + token * p.gate_row + (long long)head * p.gate_head + half * HH * p.gate_step : nullptr;
+      if (gate != nullptr && p.gate_step == 0) inv *= __fdividef(1.f, 1.f + __expf(-to_float(gate[0])));
 #pragma unroll
       for (int c = 0; c < HH; c += 8) {
         if (half * HH + c >= p.v_dim) continue;
-        if (gate != nullptr) {
+        if (gate != nullptr && p.gate_step != 0) {
           const uint4 raw = *reinterpret_cast<const uint4*>(gate + c);
           const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
@@ -569,6 +574,12 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, cons
             o[c + 2 * i] *= __fdividef(1.f, 1.f + __expf(-g.x));
             o[c + 2 * i + 1] *= __fdividef(1.f, 1.f + __expf(-g.y));
           }
+        }
+        if (p.out32 != nullptr) {
+          float4* dst32 = reinterpret_cast<float4*>(p.out32 + token * ((long long)p.n_heads * p.v_dim) + head * p.v_dim + half * HH + c);
+          dst32[0] = make_float4(o[c] * inv, o[c + 1] * inv, o[c + 2] * inv, o[c + 3] * inv);
+          dst32[1] = make_float4(o[c + 4] * inv, o[c + 5] * inv, o[c + 6] * inv, o[c + 7] * inv);
+          continue;
         }
         uint4 x;
         x.x = ta_pack(o[c] * inv, o[c + 1] * inv);
@@ -656,7 +667,7 @@ static int run_attention_prefill_tcgen05(const void* q, long long q_rows, long l
   }
   TaParams p{(__nv_bfloat16*)out, seq_start, past_len, kv_table, table_stride, table_len > 0 ? table_len : 1, status,
              n_heads, n_kv_heads, k_col, v_col, scale * 1.4426950408889634f, causal, window, keep_first, bias,
-             head_dim, v_dim, 0, nullptr, nullptr, 0, 0};
+             head_dim, v_dim, 0, nullptr, nullptr, 0, 0, 1, nullptr, 1, 0};
   BT_CHECK((v_dim == 64 || v_dim == 128) && (sigmoid || v_dim == head_dim),
            "attention_prefill_tcgen05: values of %d channels beside keys of %d are not supported", v_dim, head_dim);
   if (sigmoid) {
@@ -699,21 +710,22 @@ extern "C" int bt_sigmoid_attention_tcgen05(const void* q, long long q_rows, lon
 // Causal multi-head attention of sequences that start at position 0 with a sink and an output gate (each optional): query
 // head h at columns h * dq of the rows of `q`; keys [n_heads][rows][dq] and values [n_heads][rows][dv], rows: the step's
 // tokens; dq and dv multiples of 8, at most 128.  out: [tokens, n_heads * dv].
-extern "C" int bt_sink_attention_tcgen05_supports(int dq, int dv, long long q_row, long long gate_row, int gate_head) {
-  return dq > 0 && dv > 0 && dq <= 128 && dv <= 128 && dq % 8 == 0 && dv % 8 == 0 && q_row % 8 == 0 && gate_row % 8 == 0 &&
-         gate_head % 8 == 0;
+extern "C" int bt_sink_attention_tcgen05_supports(int dq, int dv, long long q_row, long long gate_row, int gate_head,
+                                                  int gate_step) {
+  return dq > 0 && dv > 0 && dq <= 128 && dv <= 128 && dq % 8 == 0 && dv % 8 == 0 && q_row % 8 == 0 &&
+         (gate_step == 0 || (gate_row % 8 == 0 && gate_head % 8 == 0));
 }
 
 extern "C" int bt_sink_attention_tcgen05(const void* q, long long q_row, const void* k, const void* v, long long rows,
-                                         const void* gate, long long gate_row, int gate_head, void* out, int* status,
+                                         const void* gate, long long gate_row, int gate_head, int gate_step, void* out, int* status,
                                          const int* seq_start, const int* past_len, const float* sink, int n_seqs,
                                          int max_new, int n_heads, int dq, int dv, float scale, int window,
                                          cudaStream_t stream) {
   using namespace bt;
-  BT_CHECK(bt_sink_attention_tcgen05_supports(dq, dv, q_row, gate_row, gate_head),
+  BT_CHECK(bt_sink_attention_tcgen05_supports(dq, dv, q_row, gate_row, gate_head, gate_step),
            "sink_attention_tcgen05: sizes or strides the kernel does not take (dq=%d dv=%d)", dq, dv);
   auto at16 = [](const void* ptr) { return (unsigned long long)ptr % 16 == 0; };
-  BT_CHECK(at16(q) && at16(k) && at16(v) && at16(out) && at16(gate), "sink_attention_tcgen05: operands must lie on 16-byte boundaries");
+  BT_CHECK(at16(q) && at16(k) && at16(v) && at16(out) && (gate_step == 0 || at16(gate)), "sink_attention_tcgen05: operands must lie on 16-byte boundaries");
   BT_CHECK(n_heads > 0 && n_heads <= 65535 && n_seqs <= 65535 && window >= 0 && rows >= 1 && rows * n_heads < (1ll << 31) &&
                (long long)n_heads * dq <= q_row,
            "sink_attention_tcgen05: bad sizes heads=%d sequences=%d rows=%lld", n_heads, n_seqs, rows);
@@ -725,9 +737,44 @@ extern "C" int bt_sink_attention_tcgen05(const void* q, long long q_row, const v
   if (int rc = tensor_map_2d_bf16(&vm, v, (unsigned long long)rows * n_heads, dv, dv, 64)) return rc;
   TaParams p{(__nv_bfloat16*)out, seq_start, past_len, nullptr, 0, 1, status, n_heads, n_heads, 0, 0,
              scale * 1.4426950408889634f, 1, window, 0, nullptr, dq, dv, (int)rows, sink, (const __nv_bfloat16*)gate,
-             gate_row, gate_head};
+             gate_row, gate_head, gate_step, nullptr, 1, 0};
   if (dq <= 64 && dv <= 64) return launch_ta<64, 64, false>(qm, km, vm, p, n_seqs, max_new, stream);
   if (dq <= 64) return launch_ta<64, 128, false>(qm, km, vm, p, n_seqs, max_new, stream);
   if (dv <= 64) return launch_ta<128, 64, false>(qm, km, vm, p, n_seqs, max_new, stream);
+  return launch_ta<128, 128, false>(qm, km, vm, p, n_seqs, max_new, stream);
+}
+
+// Causal attention in which every head is two maps over one value head, the maps' results left apart for a caller that
+// combines them: query map i of head h at columns (2 h + i) * pad of the rows of `q`, `pad` = 64 or 128, the channels from
+// `dim` on zero.  Keys and values come from the pages: pool [pool_pages][n_kv_heads][64][key 1 | key 2 | value] (dim, dim,
+// v_dim channels), which hold the step's own tokens too.  out: [tokens, 2 n_heads, v_dim] 32-bit.
+extern "C" int bt_two_map_attention_tcgen05_supports(int dim, int v_dim) {
+  return dim > 0 && v_dim > 0 && dim <= 128 && v_dim <= 128 && dim % 8 == 0 && v_dim % 8 == 0;
+}
+
+extern "C" int bt_two_map_attention_tcgen05(const void* q, long long rows, int pad, const void* pool, long long pool_pages,
+                                            const int* table, int table_stride, int table_len, float* out, int* status,
+                                            const int* seq_start, const int* past_len, int n_seqs, int max_new, int n_heads,
+                                            int n_kv_heads, int dim, int v_dim, float scale, cudaStream_t stream) {
+  using namespace bt;
+  BT_CHECK(bt_two_map_attention_tcgen05_supports(dim, v_dim) && (pad == 64 || pad == 128) && pad >= dim,
+           "two_map_attention_tcgen05: sizes the kernel does not take (dim=%d v_dim=%d pad=%d)", dim, v_dim, pad);
+  auto at16 = [](const void* ptr) { return (unsigned long long)ptr % 16 == 0; };
+  BT_CHECK(at16(q) && at16(pool) && at16(out), "two_map_attention_tcgen05: operands must lie on 16-byte boundaries");
+  BT_CHECK(n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0 && n_heads <= 32767 && n_seqs <= 65535 && rows >= 1 &&
+               pool_pages >= 1 && table_len >= 1 && pool_pages * n_kv_heads * 64 < (1ll << 31),
+           "two_map_attention_tcgen05: bad sizes heads=%d key heads=%d sequences=%d rows=%lld", n_heads, n_kv_heads, n_seqs, rows);
+  if (n_seqs == 0 || max_new == 0) return 0;
+  CUtensorMap qm, km, vm;
+  const unsigned long long pool_rows = (unsigned long long)pool_pages * n_kv_heads * 64, row = 2ull * dim + v_dim;
+  const unsigned long long q_cols = 2ull * n_heads * pad;
+  if (int rc = tensor_map_2d_bf16(&qm, q, (unsigned long long)rows, q_cols, q_cols, 64)) return rc;
+  if (int rc = tensor_map_2d_bf16(&km, pool, pool_rows, 2ull * dim, row, 64)) return rc;
+  if (int rc = tensor_map_2d_bf16(&vm, (const __nv_bfloat16*)pool + 2 * dim, pool_rows, v_dim, row, 64)) return rc;
+  TaParams p{nullptr, seq_start, past_len, table, table_stride, table_len, status, 2 * n_heads, n_kv_heads, 0, 0,
+             scale * 1.4426950408889634f, 1, 0, 0, nullptr, pad, v_dim, 0, nullptr, nullptr, 0, 0, 1, out, 2, dim};
+  if (pad == 64 && v_dim <= 64) return launch_ta<64, 64, false>(qm, km, vm, p, n_seqs, max_new, stream);
+  if (pad == 64) return launch_ta<64, 128, false>(qm, km, vm, p, n_seqs, max_new, stream);
+  if (v_dim <= 64) return launch_ta<128, 64, false>(qm, km, vm, p, n_seqs, max_new, stream);
   return launch_ta<128, 128, false>(qm, km, vm, p, n_seqs, max_new, stream);
 }

@@ -1,4 +1,5 @@
-// Per-head products on tensor cores (bfloat16): out[t, h, :] = a[t, h, :] @ W[h] (* sigmoid(gate[t, h, :])).
+// Per-head products on tensor cores (bfloat16): out[t, h, :] = a[t, h, :] @ W[h] (* sigmoid(gate[t, h, :])); with
+// gate_step 0 the gate is one number a head.
 // A block takes 64 tokens x 64 output columns of one head: four warps of 16 tokens each, K in pieces of 64 that pass
 // through shared memory (rows an odd number of 16-byte pieces apart, so ldmatrix meets no bank twice); W[h] is [K, N]
 // with N contiguous, read as the products' second operand through ldmatrix.trans.  Sums are 32-bit.
@@ -12,7 +13,7 @@ __global__ void __launch_bounds__(128)
 head_linear_mma_kernel(const __nv_bfloat16* __restrict__ a, long long a_row_stride, int a_head_stride,
                        const __nv_bfloat16* __restrict__ w, __nv_bfloat16* __restrict__ out, long long out_row_stride,
                        int out_head_stride, const __nv_bfloat16* __restrict__ gate, long long gate_row_stride,
-                       int gate_head_stride, int n_tokens, int K, int N) {
+                       int gate_head_stride, int gate_step, int n_tokens, int K, int N) {
   __shared__ __align__(16) __nv_bfloat16 a_s[HL_BM * HL_LD];
   __shared__ __align__(16) __nv_bfloat16 w_s[HL_BK * HL_LD];
   pdl_trigger();
@@ -79,7 +80,8 @@ head_linear_mma_kernel(const __nv_bfloat16* __restrict__ a, long long a_row_stri
       if (c >= N) continue;
       float v0 = acc[j][2 * rr], v1 = acc[j][2 * rr + 1];
       if (gt) {
-        const float2 gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gt + c));
+        const float2 gv = gate_step ? __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gt + c))
+                                    : make_float2(to_float(gt[0]), to_float(gt[0]));
         v0 *= 1.f / (1.f + expf(-gv.x));
         v1 *= 1.f / (1.f + expf(-gv.y));
       }
@@ -91,21 +93,21 @@ head_linear_mma_kernel(const __nv_bfloat16* __restrict__ a, long long a_row_stri
 // Whether the operands lie so that the kernel's 16-byte loads and 4-byte stores are aligned.
 bool head_linear_mma_supports(const void* a, long long a_row_stride, int a_head_stride, const void* w, const void* out,
                               long long out_row_stride, int out_head_stride, const void* gate, long long gate_row_stride,
-                              int gate_head_stride, int K, int N) {
+                              int gate_head_stride, int gate_step, int K, int N) {
   auto at = [](const void* p, int bytes) { return ((unsigned long long)p % bytes) == 0; };
   return K % 8 == 0 && N % 8 == 0 && at(a, 16) && a_row_stride % 8 == 0 && a_head_stride % 8 == 0 && at(w, 16) &&
          at(out, 4) && out_row_stride % 2 == 0 && out_head_stride % 2 == 0 &&
-         (gate == nullptr || (at(gate, 4) && gate_row_stride % 2 == 0 && gate_head_stride % 2 == 0));
+         (gate == nullptr || gate_step == 0 || (at(gate, 4) && gate_row_stride % 2 == 0 && gate_head_stride % 2 == 0));
 }
 
 int launch_head_linear_mma(const __nv_bfloat16* a, long long a_row_stride, int a_head_stride, const __nv_bfloat16* w,
                            __nv_bfloat16* out, long long out_row_stride, int out_head_stride, const __nv_bfloat16* gate,
-                           long long gate_row_stride, int gate_head_stride, int n_tokens, int n_heads, int K, int N,
+                           long long gate_row_stride, int gate_head_stride, int gate_step, int n_tokens, int n_heads, int K, int N,
                            cudaStream_t stream) {
   BT_CHECK(n_heads <= 65535 && (N + HL_BN - 1) / HL_BN <= 65535, "head_linear: %d heads or %d columns are too many", n_heads, N);
   const dim3 grid((n_tokens + HL_BM - 1) / HL_BM, n_heads, (N + HL_BN - 1) / HL_BN), block(128);
   BT_PDL_OK("head_linear_mma", launch_pdl(head_linear_mma_kernel, grid, block, 0, stream, 1, a, a_row_stride, a_head_stride,
-                                          w, out, out_row_stride, out_head_stride, gate, gate_row_stride, gate_head_stride,
+                                          w, out, out_row_stride, out_head_stride, gate, gate_row_stride, gate_head_stride, gate_step,
                                           n_tokens, K, N));
   return 0;
 }

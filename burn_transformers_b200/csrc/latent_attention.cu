@@ -33,10 +33,10 @@ int launch_latent_attention_mma(const __nv_bfloat16* q, long long q_row_stride, 
 // per-head products on tensor cores for bfloat16 (head_linear_mma.cu)
 bool head_linear_mma_supports(const void* a, long long a_row_stride, int a_head_stride, const void* w, const void* out,
                               long long out_row_stride, int out_head_stride, const void* gate, long long gate_row_stride,
-                              int gate_head_stride, int K, int N);
+                              int gate_head_stride, int gate_step, int K, int N);
 int launch_head_linear_mma(const __nv_bfloat16* a, long long a_row_stride, int a_head_stride, const __nv_bfloat16* w,
                            __nv_bfloat16* out, long long out_row_stride, int out_head_stride, const __nv_bfloat16* gate,
-                           long long gate_row_stride, int gate_head_stride, int n_tokens, int n_heads, int K, int N,
+                           long long gate_row_stride, int gate_head_stride, int gate_step, int n_tokens, int n_heads, int K, int N,
                            cudaStream_t stream);
 
 // ---- filing the latent ------------------------------------------------------------------------------------------
@@ -97,13 +97,13 @@ latent_gather_kernel(const T* __restrict__ pool, const int* __restrict__ positio
 // ---- per-head products ------------------------------------------------------------------------------------------
 
 // out[t, h, j] = sum_k a[t, h, k] * W[h][k][j]   (* sigmoid(gate[t, h, j]) if gate)
-// a: rows `a_row_stride` apart, head h at a_head_stride * h; out and gate likewise.  A block takes TM tokens of one
+// a: rows `a_row_stride` apart, head h at a_head_stride * h; out and gate likewise (gate_step 0: one gate a head).  A block takes TM tokens of one
 // head; a thread owns output columns j, j + blockDim, ... and keeps TM sums per column.
 template <typename T, int TM>
 __global__ void __launch_bounds__(128)
 head_linear_kernel(const T* __restrict__ a, long long a_row_stride, int a_head_stride, const T* __restrict__ w,
                    T* __restrict__ out, long long out_row_stride, int out_head_stride, const T* __restrict__ gate,
-                   long long gate_row_stride, int gate_head_stride, int n_tokens, int K, int N) {
+                   long long gate_row_stride, int gate_head_stride, int gate_step, int n_tokens, int K, int N) {
   extern __shared__ float a_s[];  // [TM][K]
   pdl_trigger();
   pdl_wait();
@@ -129,7 +129,7 @@ head_linear_kernel(const T* __restrict__ a, long long a_row_stride, int a_head_s
       if (t0 + m >= n_tokens) break;
       float v = acc[m];
       if (gate) {
-        const float g = to_float(gate[(long long)(t0 + m) * gate_row_stride + (long long)h * gate_head_stride + j]);
+        const float g = to_float(gate[(long long)(t0 + m) * gate_row_stride + (long long)h * gate_head_stride + j * gate_step]);
         v *= 1.f / (1.f + expf(-g));
       }
       out[(long long)(t0 + m) * out_row_stride + (long long)h * out_head_stride + j] = from_float<T>(v);
@@ -387,14 +387,14 @@ static int launch_latent_merge(const float* part, T* out, long long out_row_stri
 template <typename T>
 static int launch_head_linear(const T* a, long long a_row_stride, int a_head_stride, const T* w, T* out,
                               long long out_row_stride, int out_head_stride, const T* gate, long long gate_row_stride,
-                              int gate_head_stride, int n_tokens, int n_heads, int K, int N, cudaStream_t stream) {
+                              int gate_head_stride, int gate_step, int n_tokens, int n_heads, int K, int N, cudaStream_t stream) {
   constexpr int TM = 8;
   const size_t smem = (size_t)TM * K * sizeof(float);
   BT_CHECK(smem <= 48 * 1024, "head_linear: K = %d is more than the kernel's rows of shared memory hold", K);
   const dim3 grid((n_tokens + TM - 1) / TM, n_heads), block(128);
   BT_PDL_OK("head_linear", launch_pdl(head_linear_kernel<T, TM>, grid, block, smem, stream, 1, a, a_row_stride,
                                       a_head_stride, w, out, out_row_stride, out_head_stride, gate, gate_row_stride,
-                                      gate_head_stride, n_tokens, K, N));
+                                      gate_head_stride, gate_step, n_tokens, K, N));
   return 0;
 }
 
@@ -444,26 +444,26 @@ extern "C" int bt_latent_gather(const void* pool, const int* positions, const in
 
 extern "C" int bt_head_linear(const void* a, long long a_row_stride, int a_head_stride, const void* w, void* out,
                               long long out_row_stride, int out_head_stride, const void* gate, long long gate_row_stride,
-                              int gate_head_stride, int n_tokens, int n_heads, int K, int N, int tensor_cores,
+                              int gate_head_stride, int gate_step, int n_tokens, int n_heads, int K, int N, int tensor_cores,
                               int dtype, cudaStream_t stream) {
   using namespace bt;
   BT_CHECK(n_heads > 0 && K > 0 && N > 0, "head_linear: bad sizes heads=%d K=%d N=%d", n_heads, K, N);
   if (n_tokens == 0) return 0;
   if (dtype == kBF16 && tensor_cores &&
       head_linear_mma_supports(a, a_row_stride, a_head_stride, w, out, out_row_stride, out_head_stride, gate,
-                               gate_row_stride, gate_head_stride, K, N))
+                               gate_row_stride, gate_head_stride, gate_step, K, N))
     return launch_head_linear_mma((const __nv_bfloat16*)a, a_row_stride, a_head_stride, (const __nv_bfloat16*)w,
                                   (__nv_bfloat16*)out, out_row_stride, out_head_stride, (const __nv_bfloat16*)gate,
-                                  gate_row_stride, gate_head_stride, n_tokens, n_heads, K, N, stream);
+                                  gate_row_stride, gate_head_stride, gate_step, n_tokens, n_heads, K, N, stream);
   if (dtype == kF32)
     return launch_head_linear<float>((const float*)a, a_row_stride, a_head_stride, (const float*)w, (float*)out,
                                      out_row_stride, out_head_stride, (const float*)gate, gate_row_stride,
-                                     gate_head_stride, n_tokens, n_heads, K, N, stream);
+                                     gate_head_stride, gate_step, n_tokens, n_heads, K, N, stream);
   if (dtype == kBF16)
     return launch_head_linear<__nv_bfloat16>((const __nv_bfloat16*)a, a_row_stride, a_head_stride,
                                              (const __nv_bfloat16*)w, (__nv_bfloat16*)out, out_row_stride,
                                              out_head_stride, (const __nv_bfloat16*)gate, gate_row_stride,
-                                             gate_head_stride, n_tokens, n_heads, K, N, stream);
+                                             gate_head_stride, gate_step, n_tokens, n_heads, K, N, stream);
   return fail("head_linear: unknown dtype %d", dtype);
 }
 

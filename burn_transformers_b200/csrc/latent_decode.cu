@@ -129,7 +129,7 @@ template <typename T>
 __global__ void __launch_bounds__(LD_THREADS)
 latent_decode_finish_kernel(const float* __restrict__ part, const T* __restrict__ mixed_latent, int n_splits,
                             const T* __restrict__ uv,               // [heads][rank][vdim]
-                            const T* __restrict__ gate, long long gate_row_stride, T* __restrict__ out,
+                            const T* __restrict__ gate, long long gate_row_stride, int gate_per_head, T* __restrict__ out,
                             long long out_row_stride, int n_heads, int rank, int vdim) {
   extern __shared__ float sm[];      // [rank] the weighted sum of latents, then [LD_MAX_SPLITS] the splits' weights
   float* o_s = sm;
@@ -185,7 +185,7 @@ latent_decode_finish_kernel(const float* __restrict__ part, const T* __restrict_
     float acc = wide ? y_s[j] : 0.f;
     if (!wide)
       for (int r = 0; r < rank; ++r) acc = fmaf(o_s[r], to_float(w[(long long)r * vdim + j]), acc);
-    if (gate) acc *= 1.f / (1.f + expf(-to_float(gate[(long long)t * gate_row_stride + (long long)h * vdim + j])));
+    if (gate) acc *= 1.f / (1.f + expf(-to_float(gate[(long long)t * gate_row_stride + (gate_per_head ? h : (long long)h * vdim + j)])));
     out[(long long)t * out_row_stride + (long long)h * vdim + j] = from_float<T>(acc);
   }
 }
@@ -231,7 +231,7 @@ extern "C" int bt_latent_decode_prep(const void* proj, long long row_stride, int
 }
 
 extern "C" int bt_latent_decode_finish(const float* part, const void* mixed_latent, int n_splits, const void* uv,
-                                       const void* gate, long long gate_row_stride, void* out, long long out_row_stride,
+                                       const void* gate, long long gate_row_stride, int gate_per_head, void* out, long long out_row_stride,
                                        int n_tokens, int n_heads, int rank, int vdim, int dtype, cudaStream_t stream) {
   using namespace bt;
   BT_CHECK(n_heads > 0 && n_heads <= 65535 && rank > 0 && rank <= 8192 && vdim > 0 && n_splits >= 1 &&
@@ -243,12 +243,12 @@ extern "C" int bt_latent_decode_finish(const float* part, const void* mixed_late
   if (dtype == kF32)
     BT_PDL_OK("latent_decode_finish", launch_pdl(latent_decode_finish_kernel<float>, grid, block, smem, stream, 1, part,
                                                  (const float*)mixed_latent, n_splits, (const float*)uv, (const float*)gate,
-                                                 gate_row_stride, (float*)out, out_row_stride, n_heads, rank, vdim));
+                                                 gate_row_stride, gate_per_head, (float*)out, out_row_stride, n_heads, rank, vdim));
   else if (dtype == kBF16)
     BT_PDL_OK("latent_decode_finish",
               launch_pdl(latent_decode_finish_kernel<__nv_bfloat16>, grid, block, smem, stream, 1, part,
                          (const __nv_bfloat16*)mixed_latent, n_splits, (const __nv_bfloat16*)uv, (const __nv_bfloat16*)gate,
-                         gate_row_stride, (__nv_bfloat16*)out, out_row_stride, n_heads, rank, vdim));
+                         gate_row_stride, gate_per_head, (__nv_bfloat16*)out, out_row_stride, n_heads, rank, vdim));
   else
     return fail("latent_decode_finish: unknown dtype %d", dtype);
   return 0;

@@ -7,7 +7,7 @@
 //     through distributed shared memory in a fixed order (rank 0, 1, ...), so the result is deterministic and
 //     needs neither atomics nor scratch memory;
 //   * optionally the rows (at most 16) are LayerNorm-ed on the way in (32-bit statistics over the full row,
-//     two passes), which saves a kernel and a round trip of the normalised rows;
+//     two passes) or RMS-normed (one pass), which saves a kernel and a round trip of the normalised rows;
 //   * the weight panel is requested before the kernel waits for its predecessor (programmatic dependent
 //     launch), so weights stream while the previous kernel is still finishing;
 //   * the epilogue adds the bias, applies GELU, adds the 32-bit residual and writes 32-bit or bfloat16.
@@ -36,6 +36,7 @@ struct SkinnyParams {
   const float* residual;       // [M, N] 32-bit or null (may be `out`)
   void* out;                   // [M, N] 32-bit or bfloat16
   int M, N, K, k_slice, act, out_is_f32;
+  int rms;                     // the fused norm subtracts no mean: x / sqrt(mean(x^2) + eps) * gamma
 };
 
 __device__ __forceinline__ void ldmatrix_x4(unsigned (&r)[4], const void* p) {
@@ -118,7 +119,7 @@ linear_skinny_kernel(SkinnyParams p) {
       const bool live = r < p.M;
       const float* src = p.x32 + (long long)(live ? (p.rows ? p.rows[r] : r) : 0) * p.K;
       float s = 0.f;
-      if (live)
+      if (live && !p.rms)
         for (int c = li * 4; c < p.K; c += lanes_per_row * 4) {
           const float4 v = *reinterpret_cast<const float4*>(src + c);
           s += (v.x + v.y) + (v.z + v.w);
@@ -288,12 +289,12 @@ extern "C" int bt_linear_skinny_supports(int M, int N, int K, int w_is_nk, int f
   return 1;
 }
 
-// a: bfloat16 rows, or null with (x32, gamma, beta, eps, rows) to normalise 32-bit rows on the way in.
+// a: bfloat16 rows, or null with (x32, gamma, beta, eps, rows) to normalise 32-bit rows on the way in (rms: an RMS norm).
 // split: blocks per cluster along K (1..8); 0 lets the library choose.
 extern "C" int bt_linear_skinny(const void* a, const float* x32, const int* rows, const float* gamma,
                                 const float* beta, float eps, const void* w, const float* bias,
                                 const float* residual, void* out, int M, int N, int K, int w_is_nk, int act,
-                                int out_is_f32, int split, cudaStream_t stream) {
+                                int out_is_f32, int split, int rms, cudaStream_t stream) {
   using namespace bt;
   const int fuse_ln = a == nullptr;
   BT_CHECK(bt_linear_skinny_supports(M, N, K, w_is_nk, fuse_ln), "linear_skinny: sizes M=%d N=%d K=%d are not supported", M, N, K);
@@ -313,7 +314,7 @@ extern "C" int bt_linear_skinny(const void* a, const float* x32, const int* rows
   BT_CHECK(split >= 1 && split <= 8, "linear_skinny: split %d is outside 1..8", split);
   int k_slice = ((K + split - 1) / split + 15) / 16 * 16;
   SkinnyParams p{(const __nv_bfloat16*)a, x32, rows, gamma, beta, eps, (const __nv_bfloat16*)w, bias, residual, out,
-                 M, N, K, k_slice, act, out_is_f32};
+                 M, N, K, k_slice, act, out_is_f32, rms};
   if (w_is_nk) return fuse_ln ? launch_skinny_mt<true, true>(p, split, stream) : launch_skinny_mt<true, false>(p, split, stream);
   return fuse_ln ? launch_skinny_mt<false, true>(p, split, stream) : launch_skinny_mt<false, false>(p, split, stream);
 }

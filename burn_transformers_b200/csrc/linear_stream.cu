@@ -35,6 +35,7 @@ struct StreamParams {
   const float* residual;    // [M, N] 32-bit or null (may be `out`)
   void* out;
   int M, N, K, act, out_is_f32;
+  int rms;                  // the fused norm subtracts no mean: x / sqrt(mean(x^2) + eps) * gamma
 };
 
 __device__ __forceinline__ uint4 ld_stream16(const void* p) {   // read once: do not keep in L1
@@ -98,7 +99,7 @@ linear_stream_kernel(StreamParams p) {
       if (r < p.M) {
         const float* src = p.x32 + (long long)(p.rows ? p.rows[r] : r) * p.K;
         float s = 0.f;
-        for (int c = lane * 4; c < p.K; c += 128) {
+        for (int c = lane * 4; c < p.K && !p.rms; c += 128) {
           const float4 v = *reinterpret_cast<const float4*>(src + c);
           s += (v.x + v.y) + (v.z + v.w);
         }
@@ -236,12 +237,12 @@ extern "C" int bt_linear_stream_supports(int M, int N, int K, int fuse_ln) {
   return 1;
 }
 
-// w: [N, K] bfloat16.  a: bfloat16 rows, or null with (x32, gamma, beta, eps, rows) to normalise on the way in.
+// w: [N, K] bfloat16.  a: bfloat16 rows, or null with (x32, gamma, beta, eps, rows) to normalise on the way in (rms: an RMS norm).
 // warps_k: warps of a block that split K (1, 2, 4); 0 lets the library choose.
 extern "C" int bt_linear_stream(const void* a, const float* x32, const int* rows, const float* gamma,
                                 const float* beta, float eps, const void* w, const float* bias,
                                 const float* residual, void* out, int M, int N, int K, int act, int out_is_f32,
-                                int warps_k, cudaStream_t stream) {
+                                int warps_k, int rms, cudaStream_t stream) {
   using namespace bt;
   const int fuse_ln = a == nullptr;
   BT_CHECK(bt_linear_stream_supports(M, N, K, fuse_ln), "linear_stream: sizes M=%d N=%d K=%d are not supported", M, N, K);
@@ -258,7 +259,7 @@ extern "C" int bt_linear_stream(const void* a, const float* x32, const int* rows
   }
   BT_CHECK(warps_k == 1 || warps_k == 2 || warps_k == 4, "linear_stream: warps_k %d must be 1, 2 or 4", warps_k);
   StreamParams p{(const __nv_bfloat16*)a, x32, rows, gamma, beta, eps, (const __nv_bfloat16*)w, bias, residual, out,
-                 M, N, K, act, out_is_f32};
+                 M, N, K, act, out_is_f32, rms};
   if (fuse_ln) {
     if (warps_k == 1) return launch_stream_mt<1, true>(p, stream);
     if (warps_k == 2) return launch_stream_mt<2, true>(p, stream);

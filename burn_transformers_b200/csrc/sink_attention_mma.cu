@@ -1,5 +1,5 @@
 // Causal multi-head attention of fresh prompts on tensor cores (bfloat16), with an optional per-head sink in the
-// softmax denominator and an optional sigmoid gate on the result: the plain form of the latent attention for steps in
+// softmax denominator and an optional sigmoid gate (a number a channel, or one a head: gate_step 0) on the result: the plain form of the latent attention for steps in
 // which every sequence starts at position 0, so that keys and values are the step's own rows (up-projected per head by
 // the caller).  It does dq + dv multiply-adds a key and head where the form that carries the query into the latent
 // space does 2 rank + rot.
@@ -29,6 +29,7 @@ struct SinkAttentionArgs {
   __nv_bfloat16* out;
   long long q_row, k_row, v_row, gate_row, out_row;     // elements between tokens
   int q_head, k_head, v_head, gate_head, out_head;      // elements between heads
+  int gate_step;                                        // elements between a head's gates: 1, or 0 for one gate a head
   const int* seq_start;
   const float* sink;
   int dq, dv;
@@ -236,7 +237,8 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(SinkAttentionAr
       if (c >= p.dv) continue;
       float v0 = acc[j][2 * rr] * inv, v1 = acc[j][2 * rr + 1] * inv;
       if (gt) {
-        const float2 gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gt + c));
+        const float2 gv = p.gate_step ? __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gt + c))
+                                      : make_float2(to_float(gt[0]), to_float(gt[0]));
         v0 *= 1.f / (1.f + expf(-gv.x));
         v1 *= 1.f / (1.f + expf(-gv.y));
       }
@@ -249,25 +251,25 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(SinkAttentionAr
 
 // 1 if the operands lie so that the kernel takes them: whole 16-byte pieces per head and row, at most 128 value channels.
 extern "C" int bt_sink_attention_supports(int dq, int dv, long long q_row, int q_head, long long k_row, int k_head,
-                                          long long v_row, int v_head, long long gate_row, int gate_head,
+                                          long long v_row, int v_head, long long gate_row, int gate_head, int gate_step,
                                           long long out_row, int out_head) {
   return dq > 0 && dv > 0 && dq % 8 == 0 && dv % 8 == 0 && dv <= 128 && dq <= 512 && q_row % 8 == 0 && q_head % 8 == 0 &&
-         k_row % 8 == 0 && k_head % 8 == 0 && v_row % 8 == 0 && v_head % 8 == 0 && gate_row % 2 == 0 && gate_head % 2 == 0 &&
+         k_row % 8 == 0 && k_head % 8 == 0 && v_row % 8 == 0 && v_head % 8 == 0 && (gate_step == 0 || (gate_row % 2 == 0 && gate_head % 2 == 0)) &&
          out_row % 2 == 0 && out_head % 2 == 0;
 }
 
 extern "C" int bt_sink_attention(const void* q, long long q_row, int q_head, const void* k, long long k_row, int k_head,
                                  const void* v, long long v_row, int v_head, const void* gate, long long gate_row,
-                                 int gate_head, void* out, long long out_row, int out_head, const int* seq_start,
+                                 int gate_head, int gate_step, void* out, long long out_row, int out_head, const int* seq_start,
                                  const float* sink, int n_seqs, int max_new, int n_heads, int dq, int dv, float scale,
                                  int window, int keep_first, int kv_group, int sigmoid, const float* bias,
                                  cudaStream_t stream) {
   using namespace bt;
-  BT_CHECK(bt_sink_attention_supports(dq, dv, q_row, q_head, k_row, k_head, v_row, v_head, gate_row, gate_head, out_row,
+  BT_CHECK(bt_sink_attention_supports(dq, dv, q_row, q_head, k_row, k_head, v_row, v_head, gate_row, gate_head, gate_step, out_row,
                                       out_head),
            "sink_attention: sizes or strides the kernel does not take (dq=%d dv=%d)", dq, dv);
   auto at = [](const void* ptr, int bytes) { return ((unsigned long long)ptr % bytes) == 0; };
-  BT_CHECK(at(q, 16) && at(k, 16) && at(v, 16) && at(out, 4) && (gate == nullptr || at(gate, 4)),
+  BT_CHECK(at(q, 16) && at(k, 16) && at(v, 16) && at(out, 4) && (gate == nullptr || gate_step == 0 || at(gate, 4)),
            "sink_attention: operands must lie on 16-byte boundaries");
   BT_CHECK(n_heads > 0 && n_heads <= 65535 && n_seqs <= 65535 && kv_group > 0 && n_heads % kv_group == 0 && window >= 0 &&
                keep_first >= 0,
@@ -277,7 +279,7 @@ extern "C" int bt_sink_attention(const void* q, long long q_row, int q_head, con
   p.q = (const __nv_bfloat16*)q; p.k = (const __nv_bfloat16*)k; p.v = (const __nv_bfloat16*)v;
   p.gate = (const __nv_bfloat16*)gate; p.out = (__nv_bfloat16*)out;
   p.q_row = q_row; p.k_row = k_row; p.v_row = v_row; p.gate_row = gate_row; p.out_row = out_row;
-  p.q_head = q_head; p.k_head = k_head; p.v_head = v_head; p.gate_head = gate_head; p.out_head = out_head;
+  p.q_head = q_head; p.k_head = k_head; p.v_head = v_head; p.gate_head = gate_head; p.gate_step = gate_step; p.out_head = out_head;
   p.seq_start = seq_start; p.sink = sink; p.dq = dq; p.dv = dv; p.scale = scale; p.window = window;
   p.keep_first = keep_first; p.kv_group = kv_group; p.bias = bias;
   const int dqp = (dq + 15) & ~15, dvp = (dv + 15) & ~15;

@@ -55,7 +55,7 @@ class KernelProfile:
     SKIP = ("bt_last_error", "bt_launch_count", "bt_abi_version", "bt_tensor_map", "bt_decode_flow_plan",
             "bt_decode_flow_phase_bytes", "bt_attention_decode_scratch_floats", "bt_latent_attention_scratch_floats",
             "bt_latent_attention_rows", "bt_lightning_chunked_scratch_floats", "bt_sink_attention_supports",
-            "bt_mlstm_chunked_scratch_floats", "bt_moe_tile_rows", "bt_mlstm_scan_fuses")
+            "bt_mlstm_chunked_scratch_floats", "bt_moe_tile_rows", "bt_mlstm_scan_fuses", "bt_gla_scan_fuses")
 
     def __init__(self, context_hint: int | None = None):
         self.records = []          # (name, start event, stop event, flops, bytes)
@@ -251,11 +251,11 @@ def linear_skinny_supports(m, n, k, w_is_nk, fuse_ln) -> bool:
     return _supports("bt_linear_skinny_supports", m, n, k, 1 if w_is_nk else 0, 1 if fuse_ln else 0)
 
 
-def linear_skinny(a, w, bias, out, *, m, w_is_nk=False, activation=None, residual=None, norm=None, split=0):
+def linear_skinny(a, w, bias, out, *, m, w_is_nk=False, activation=None, residual=None, norm=None, split=0, rms=False):
     """out[:m] = act(rows @ w + bias) (+ residual) for at most 64 bfloat16 rows.
 
     rows are `a` (bfloat16 [M, K]) or, when `norm` = (x32, gamma, beta, eps, row_index) is given and `a` is None,
-    LayerNorm(x32[row_index]) formed inside the kernel."""
+    LayerNorm(x32[row_index]) formed inside the kernel (with `rms` an RMS norm: no mean is taken off)."""
     n = w.shape[0] if w_is_nk else w.shape[1]
     k = w.shape[1] if w_is_nk else w.shape[0]
     _need(w, "w", torch.bfloat16, (n, k) if w_is_nk else (k, n))
@@ -288,7 +288,7 @@ def linear_skinny(a, w, bias, out, *, m, w_is_nk=False, activation=None, residua
     _check(library().bt_linear_skinny(_ptr(a if norm is None else None), _ptr(x32), _ptr(rows), _ptr(gamma), _ptr(beta),
                                       c_float(eps), _ptr(w), _ptr(bias), _ptr(residual), _ptr(out), c_int(m), c_int(n),
                                       c_int(k), c_int(1 if w_is_nk else 0), c_int(ACTIVATIONS[activation]),
-                                      c_int(1 if out.dtype == torch.float32 else 0), c_int(split), _stream()))
+                                      c_int(1 if out.dtype == torch.float32 else 0), c_int(split), c_int(1 if rms else 0), _stream()))
 
 
 def linear_mid(a, w, bias, out, *, m, activation=None, residual=None, split=0):
@@ -310,7 +310,7 @@ def linear_mid(a, w, bias, out, *, m, activation=None, residual=None, split=0):
     _linear_work(m, n, k, a, w, out)
     _check(library().bt_linear_mid(_ptr(a), _ptr(w), _ptr(bias), _ptr(residual), _ptr(out), _ptr(kernel_status(a.device)),
                                    c_int(m), c_int(n), c_int(k), c_int(ACTIVATIONS[activation]),
-                                   c_int(1 if out.dtype == torch.float32 else 0), c_int(split), _stream()))
+                                   c_int(1 if out.dtype == torch.float32 else 0), c_int(split), c_int(1 if rms else 0), _stream()))
 
 
 def linear_mid_supports(m, n, k) -> bool:
@@ -386,11 +386,11 @@ def linear_stream_supports(m, n, k, fuse_ln) -> bool:
     return _supports("bt_linear_stream_supports", m, n, k, 1 if fuse_ln else 0)
 
 
-def linear_stream(a, w, bias, out, *, m, activation=None, residual=None, norm=None, warps_k=0):
+def linear_stream(a, w, bias, out, *, m, activation=None, residual=None, norm=None, warps_k=0, rms=False):
     """out[:m] = act(rows @ w^T + bias) (+ residual) for at most 64 bfloat16 rows; w is [N, K].
 
     rows are `a` (bfloat16 [M, K]) or, when `norm` = (x32, gamma, beta, eps, row_index) is given and `a` is None,
-    LayerNorm(x32[row_index]) formed inside the kernel (at most 16 rows)."""
+    LayerNorm(x32[row_index]) formed inside the kernel (at most 16 rows; with `rms` an RMS norm: no mean is taken off)."""
     n, k = w.shape
     _need(w, "w", torch.bfloat16, (n, k))
     _need(out, "out", (torch.float32, torch.bfloat16), (None, n))
@@ -422,7 +422,7 @@ def linear_stream(a, w, bias, out, *, m, activation=None, residual=None, norm=No
     _check(library().bt_linear_stream(_ptr(a if norm is None else None), _ptr(x32), _ptr(rows), _ptr(gamma), _ptr(beta),
                                       c_float(eps), _ptr(w), _ptr(bias), _ptr(residual), _ptr(out), c_int(m), c_int(n),
                                       c_int(k), c_int(ACTIVATIONS[activation]),
-                                      c_int(1 if out.dtype == torch.float32 else 0), c_int(warps_k), _stream()))
+                                      c_int(1 if out.dtype == torch.float32 else 0), c_int(warps_k), c_int(1 if rms else 0), _stream()))
 
 
 def kv_append(proj, k_offset, v_offset, positions, token_seq, ctx_len, table, table_len, k_pool, v_pool,
@@ -679,18 +679,27 @@ def _head_view(t, name, n_heads, width):
     return t.stride(0), t.stride(1)
 
 
+def _gate_view(t, n_heads, width):
+    """(row stride, head stride, channel step) of a gate [tokens, heads, width]: a number a channel (step 1) or one a head
+    (a view expanded from [tokens, heads, 1]: step 0)."""
+    if t.dim() == 3 and t.stride(2) == 0 and t.shape[1] == n_heads and t.shape[2] == width and t.is_cuda:
+        return t.stride(0), t.stride(1), 0
+    return (*_head_view(t, "gate", n_heads, width), 1)
+
+
 def head_linear(a, w, out, *, n_tokens, gate=None, tensor_cores=True):
     """out[t, h, :] = a[t, h, :] @ w[h]  (times sigmoid(gate[t, h, :]) if `gate`), sums in 32-bit.
 
-    a: view [tokens, heads, K]; w: [heads, K, N] contiguous; out and gate: views [tokens, heads, N].  bfloat16 operands
+    a: view [tokens, heads, K]; w: [heads, K, N] contiguous; out and gate: views [tokens, heads, N] (a gate of one number
+    a head: expanded from [tokens, heads, 1]).  bfloat16 operands
     that lie on 16-byte boundaries with K and N multiples of 8 run on tensor cores (`tensor_cores=False`: never)."""
     n_heads, k, n = w.shape
     _need(w, "w", (torch.float32, torch.bfloat16), (n_heads, k, n))
     a_rs, a_hs = _head_view(a, "a", n_heads, k)
     o_rs, o_hs = _head_view(out, "out", n_heads, n)
-    g_rs = g_hs = 0
+    g_rs = g_hs = g_step = 0
     if gate is not None:
-        g_rs, g_hs = _head_view(gate, "gate", n_heads, n)
+        g_rs, g_hs, g_step = _gate_view(gate, n_heads, n)
     for name, t in (("a", a), ("out", out)) + ((("gate", gate),) if gate is not None else ()):
         if t.dtype is not w.dtype:
             raise ShapeError(f"head_linear: {name} is {t.dtype}, the weights are {w.dtype}")
@@ -698,7 +707,7 @@ def head_linear(a, w, out, *, n_tokens, gate=None, tensor_cores=True):
             raise ShapeError(f"head_linear: {n_tokens} tokens asked of {name}[{t.shape[0]}]")
     _work(2.0 * n_tokens * n_heads * k * n, (n_tokens * n_heads * (k + n) + n_heads * k * n) * w.element_size())
     _check(library().bt_head_linear(_ptr(a), c_longlong(a_rs), c_int(a_hs), _ptr(w), _ptr(out), c_longlong(o_rs),
-                                    c_int(o_hs), _ptr(gate), c_longlong(g_rs), c_int(g_hs), c_int(n_tokens),
+                                    c_int(o_hs), _ptr(gate), c_longlong(g_rs), c_int(g_hs), c_int(g_step), c_int(n_tokens),
                                     c_int(n_heads), c_int(k), c_int(n), c_int(1 if tensor_cores else 0),
                                     c_int(_code(w.dtype)), _stream()))
 
@@ -1063,9 +1072,9 @@ def _sink_attention_strides(q, k, v, gate, out):
     heads = q.shape[1]
     strides = []
     for name, t, width in (("q", q, q.shape[2]), ("k", k, q.shape[2]), ("v", v, v.shape[2]),
-                           ("gate", gate, v.shape[2]), ("out", out, v.shape[2])):
-        strides.append((0, 0) if t is None else _head_view(t, name, heads, width))
-    return strides
+                           ("out", out, v.shape[2])):
+        strides.append(_head_view(t, name, heads, width))
+    return (*strides, (0, 0, 0) if gate is None else _gate_view(gate, heads, v.shape[2]))
 
 
 def sink_attention_supports(q, k, v, gate, out) -> bool:
@@ -1073,12 +1082,12 @@ def sink_attention_supports(q, k, v, gate, out) -> bool:
     channels, operands on 16-byte boundaries."""
     if any(t is not None and t.dtype is not torch.bfloat16 for t in (q, k, v, gate, out)):
         return False
-    (qr, qh), (kr, kh), (vr, vh), (gr, gh), (orow, oh) = _sink_attention_strides(q, k, v, gate, out)
-    if any(t.data_ptr() % 16 for t in (q, k, v)) or out.data_ptr() % 4 or (gate is not None and gate.data_ptr() % 4):
+    (qr, qh), (kr, kh), (vr, vh), (orow, oh), (gr, gh, gs) = _sink_attention_strides(q, k, v, gate, out)
+    if any(t.data_ptr() % 16 for t in (q, k, v)) or out.data_ptr() % 4 or (gs and gate.data_ptr() % 4):
         return False
     return bool(library().bt_sink_attention_supports(c_int(q.shape[2]), c_int(v.shape[2]), c_longlong(qr), c_int(qh),
                                                      c_longlong(kr), c_int(kh), c_longlong(vr), c_int(vh), c_longlong(gr),
-                                                     c_int(gh), c_longlong(orow), c_int(oh)))
+                                                     c_int(gh), c_int(gs), c_longlong(orow), c_int(oh)))
 
 
 def sink_attention_tcgen05_supports(q, k, v, gate, out) -> bool:
@@ -1086,19 +1095,19 @@ def sink_attention_tcgen05_supports(q, k, v, gate, out) -> bool:
     by side in a row, keys and values head by head ([heads, tokens, channels] in memory), out contiguous."""
     if any(t is not None and t.dtype is not torch.bfloat16 for t in (q, k, v, gate, out)):
         return False
-    (qr, qh), (kr, kh), (vr, vh), (gr, gh), (orow, oh) = _sink_attention_strides(q, k, v, gate, out)
+    (qr, qh), (kr, kh), (vr, vh), (orow, oh), (gr, gh, gs) = _sink_attention_strides(q, k, v, gate, out)
     n, heads, dq, dv = q.shape[0], q.shape[1], q.shape[2], v.shape[2]
     if k.shape[0] != n or v.shape[0] != n or (qh, kr, kh, vr, vh, orow, oh) != (dq, dq, n * dq, dv, n * dv, heads * dv, dv):
         return False
-    if any(t is not None and t.data_ptr() % 16 for t in (q, k, v, gate, out)):
+    if any(t.data_ptr() % 16 for t in (q, k, v, out)) or (gs and gate.data_ptr() % 16):
         return False
-    return _supports("bt_sink_attention_tcgen05_supports", dq, dv, qr, gr, gh)
+    return _supports("bt_sink_attention_tcgen05_supports", dq, dv, qr, gr, gh, gs)
 
 
 def sink_attention(q, k, v, out, seq_start, *, n_seqs, max_new, scale, sink=None, gate=None, window=0, past_len=None, impl=None):
     """Causal multi-head attention of sequences that start at position 0, on tensor cores (bfloat16): token t of a
     sequence sees the sequence's tokens up to itself.  q, k: views [tokens, heads, dq]; v, out, gate: views
-    [tokens, heads, dv].  `sink` [heads] adds exp(sink_h) to head h's softmax denominator; `gate` multiplies the result by
+    [tokens, heads, dv] (a gate of one number a head: expanded from [tokens, heads, 1]).  `sink` [heads] adds exp(sink_h) to head h's softmax denominator; `gate` multiplies the result by
     sigmoid(gate).  Scores, softmax and sums are 32-bit.  With `past_len` (int32, zeros: one a sequence) and views that
     sink_attention_tcgen05_supports takes, both products are tcgen05.mma with the scores in tensor memory
     (csrc/attention_prefill_tcgen05.cu), else mma.sync (csrc/sink_attention_mma.cu); `impl` ("tcgen05", "mma") asks for one
@@ -1111,7 +1120,7 @@ def sink_attention(q, k, v, out, seq_start, *, n_seqs, max_new, scale, sink=None
         raise ShapeError("sink_attention: the kernel does not take these views (see sink_attention_supports)")
     if sink is not None:
         _need(sink, "sink", torch.float32, (heads,))
-    (qr, qh), (kr, kh), (vr, vh), (gr, gh), (orow, oh) = _sink_attention_strides(q, k, v, gate, out)
+    (qr, qh), (kr, kh), (vr, vh), (orow, oh), (gr, gh, gs) = _sink_attention_strides(q, k, v, gate, out)
     if _PROFILE is not None:
         ctx = float(_PROFILE.context_hint or 0)
         seen = ctx / 2 if not window or window >= ctx else window - window * window / (2.0 * ctx)
@@ -1119,13 +1128,13 @@ def sink_attention(q, k, v, out, seq_start, *, n_seqs, max_new, scale, sink=None
     if impl == "tcgen05":
         _need(past_len, "past_len", torch.int32)
         _check(library().bt_sink_attention_tcgen05(_ptr(q), c_longlong(qr), _ptr(k), _ptr(v), c_longlong(q.shape[0]), _ptr(gate),
-                                                   c_longlong(gr), c_int(gh), _ptr(out), _ptr(kernel_status(q.device)),
+                                                   c_longlong(gr), c_int(gh), c_int(gs), _ptr(out), _ptr(kernel_status(q.device)),
                                                    _ptr(seq_start), _ptr(past_len), _ptr(sink), c_int(n_seqs), c_int(max_new),
                                                    c_int(heads), c_int(dq), c_int(dv), c_float(scale), c_int(window),
                                                    _stream()))
         return
     _check(library().bt_sink_attention(_ptr(q), c_longlong(qr), c_int(qh), _ptr(k), c_longlong(kr), c_int(kh), _ptr(v),
-                                       c_longlong(vr), c_int(vh), _ptr(gate), c_longlong(gr), c_int(gh), _ptr(out),
+                                       c_longlong(vr), c_int(vh), _ptr(gate), c_longlong(gr), c_int(gh), c_int(gs), _ptr(out),
                                        c_longlong(orow), c_int(oh), _ptr(seq_start), _ptr(sink), c_int(n_seqs),
                                        c_int(max_new), c_int(heads), c_int(dq), c_int(dv), c_float(scale), c_int(window),
                                        c_int(0), c_int(1), c_int(0), c_void_p(0), _stream()))
@@ -1169,7 +1178,7 @@ def latent_decode_finish(uv_heads, out, *, n_tokens, n_splits, scratch=None, mix
     """For steps of few tokens, in one launch: joins the `n_splits` partial results of latent_attention(merge=False) in
     `scratch` (or reads `mixed_latent` [tokens, heads * rank] when there was one split), multiplies each head's weighted
     latent by uv_heads[h] ([heads, rank, vdim]) and by sigmoid(gate).  out: [tokens, heads * vdim]; gate: a view
-    [tokens, heads * vdim] with contiguous channels."""
+    [tokens, heads * vdim] (a number a channel) or [tokens, heads] (one a head) with contiguous channels."""
     n_heads, rank, vdim = uv_heads.shape
     _need(uv_heads, "uv_heads", (torch.float32, torch.bfloat16), (n_heads, rank, vdim))
     _need(out, "out", uv_heads.dtype, (None, n_heads * vdim))
@@ -1179,15 +1188,17 @@ def latent_decode_finish(uv_heads, out, *, n_tokens, n_splits, scratch=None, mix
             raise ShapeError(f"latent_decode_finish: {n_splits} splits leave {need} floats of partial results")
     else:
         _need(mixed_latent, "mixed_latent", uv_heads.dtype, (None, n_heads * rank))
-    g_rs = 0
+    g_rs = per_head = 0
     if gate is not None:
-        if gate.dim() != 2 or gate.shape[1] != n_heads * vdim or gate.stride(1) != 1 or gate.dtype is not uv_heads.dtype:
-            raise ShapeError("latent_decode_finish: gate must be a view [tokens, heads * vdim] of the weights' type")
-        g_rs = gate.stride(0)
+        if (gate.dim() != 2 or gate.shape[1] not in (n_heads, n_heads * vdim) or gate.stride(1) != 1
+                or gate.dtype is not uv_heads.dtype):
+            raise ShapeError("latent_decode_finish: gate must be a view [tokens, heads * vdim] or [tokens, heads] of the "
+                             "weights' type")
+        g_rs, per_head = gate.stride(0), int(gate.shape[1] == n_heads)
     _check(library().bt_latent_decode_finish(_ptr(scratch if n_splits > 1 else None),
                                              _ptr(mixed_latent if n_splits == 1 else None), c_int(n_splits), _ptr(uv_heads),
-                                             _ptr(gate), c_longlong(g_rs), _ptr(out), c_longlong(out.shape[1]),
-                                             c_int(n_tokens), c_int(n_heads), c_int(rank), c_int(vdim),
+                                             _ptr(gate), c_longlong(g_rs), c_int(per_head), _ptr(out),
+                                             c_longlong(out.shape[1]), c_int(n_tokens), c_int(n_heads), c_int(rank), c_int(vdim),
                                              c_int(_code(uv_heads.dtype)), _stream()))
 
 
@@ -1571,7 +1582,7 @@ def sigmoid_attention_prompt_supports(q, k, v, out) -> bool:
         return False
     return bool(library().bt_sink_attention_supports(c_int(q.shape[2]), c_int(v.shape[2]), c_longlong(qr), c_int(qh),
                                                      c_longlong(kr), c_int(kh), c_longlong(vr), c_int(vh), c_longlong(0),
-                                                     c_int(0), c_longlong(orow), c_int(oh)))
+                                                     c_int(0), c_int(0), c_longlong(orow), c_int(oh)))
 
 
 def sigmoid_attention_prompt(q, k, v, out, seq_start, *, n_seqs, max_new, scale, bias=None, window=0, keep_first=0):
@@ -1591,7 +1602,7 @@ def sigmoid_attention_prompt(q, k, v, out, seq_start, *, n_seqs, max_new, scale,
         _work(2.0 * q.shape[0] * heads * seen * (q.shape[2] + v.shape[2]),
               2.0 * q.shape[0] * (heads * (q.shape[2] + v.shape[2]) + groups * (q.shape[2] + v.shape[2])))
     _check(library().bt_sink_attention(_ptr(q), c_longlong(qr), c_int(qh), _ptr(k), c_longlong(kr), c_int(kh), _ptr(v),
-                                       c_longlong(vr), c_int(vh), c_void_p(0), c_longlong(0), c_int(0), _ptr(out),
+                                       c_longlong(vr), c_int(vh), c_void_p(0), c_longlong(0), c_int(0), c_int(0), _ptr(out),
                                        c_longlong(orow), c_int(oh), _ptr(seq_start), c_void_p(0), c_int(n_seqs),
                                        c_int(max_new), c_int(heads), c_int(q.shape[2]), c_int(v.shape[2]), c_float(scale),
                                        c_int(window), c_int(keep_first), c_int(heads // groups), c_int(1), _ptr(bias),
@@ -1624,3 +1635,168 @@ def sigmoid_attention(q, out, pool, table, table_len, seq_start, past_len, *, n_
         c_int(PAGE_SIZE), _ptr(seq_start), _ptr(past_len), _ptr(bias), _ptr(out), c_longlong(out.shape[1]), c_int(n_seqs),
         c_int(max_new), c_int(n_heads), c_int(n_kv_heads), c_int(dim), c_int(vdim), c_float(scale), c_int(window),
         c_int(keep_first), c_int(_code(q.dtype)), _stream()))
+
+
+# ---- differential attention (csrc/differential_attention.cu) and gated linear attention (csrc/gla.cu) -------------------
+
+MAX_SPLITS = 64          # blocks a row's keys are shared among at most
+
+
+def differential_prep(proj, conv, state, slots, seq_start, token_seq, positions, q_weight, k_weight, eps, inv_freq, rot_dims,
+                      rot_size, table, table_len, pool, q_out, *, n_tokens, n_seqs, max_new, n_heads, n_kv_heads, dim, vdim):
+    """Per token of rows [q | k | v] (2 heads dim, 2 kv_heads dim, kv_heads vdim channels) of `proj`: the causal convolution
+    (`conv` [taps, channels] 32-bit, `state` [slots, taps - 1, channels] with the sequences' last inputs, moved on), for every
+    map of a query or key head the division by its root mean square and the weight (`q_weight`, `k_weight` [dim] or None)
+    and the turn of the first `rot_dims` channels (neighbours paired, sine and cosine times `rot_size`); queries into q_out
+    [tokens, 2 heads * pad] (zeros behind a map's channels), [key 1 | key 2 | value] into the token's row of `pool`."""
+    _need(proj, "proj", (torch.float32, torch.bfloat16))
+    channels = 2 * (n_heads + n_kv_heads) * dim + n_kv_heads * vdim
+    taps = conv.shape[0]
+    _need(conv, "conv", torch.float32, (taps, channels))
+    _need(pool, "pool", proj.dtype, (None, n_kv_heads, PAGE_SIZE, 2 * dim + vdim))
+    _need(q_out, "q_out", proj.dtype)
+    _need(inv_freq, "inv_freq", torch.float32)
+    if taps > 1:
+        _need(state, "state", torch.float32, (None, taps - 1, channels))
+    for name, w in (("q_weight", q_weight), ("k_weight", k_weight)):
+        if w is not None:
+            _need(w, name, torch.float32, (dim,))
+    pad, rest = divmod(q_out.shape[1], 2 * n_heads)
+    if (proj.shape[1] < channels or min(proj.shape[0], q_out.shape[0]) < n_tokens or rest or pad < dim
+            or inv_freq.numel() < rot_dims // 2 or (q_weight is None) != (k_weight is None)):
+        raise ShapeError("differential_prep: rows, channels, weights or frequencies do not fit the sizes")
+    _work(0.0, float(n_tokens) * (2 * channels + 2 * n_heads * (pad - dim)) * proj.element_size())
+    _check(library().bt_differential_prep(
+        _ptr(proj), c_longlong(proj.shape[1]), _ptr(conv), _ptr(state), _ptr(slots), _ptr(seq_start), _ptr(token_seq),
+        _ptr(positions), _ptr(q_weight), _ptr(k_weight), c_float(eps), _ptr(inv_freq), c_int(rot_dims), c_float(rot_size),
+        c_int(taps), _ptr(table), c_int(table.shape[1]), c_int(table_len), c_int(PAGE_SIZE), _ptr(pool), _ptr(q_out), c_int(pad),
+        c_int(n_tokens), c_int(n_seqs), c_int(max_new), c_int(n_heads), c_int(n_kv_heads), c_int(dim), c_int(vdim),
+        c_int(_code(proj.dtype)), _stream()))
+
+
+def two_map_attention_floats(n_tokens, n_heads, vdim, n_splits) -> int:
+    """Floats of `out` of two_map_attention."""
+    return n_tokens * 2 * n_heads * (n_splits * (vdim + 2) if n_splits > 1 else vdim)
+
+
+def two_map_attention_tcgen05_supports(dim, vdim) -> bool:
+    return _supports("bt_two_map_attention_tcgen05_supports", dim, vdim)
+
+
+def _two_map_work(n_tokens, n_heads, n_kv_heads, dim, vdim, elem, decode):
+    if _PROFILE is not None:
+        ctx = float(_PROFILE.context_hint or 0)
+        seen = ctx if decode else ctx / 2
+        kv = n_tokens * seen if decode else n_tokens
+        _work(4.0 * n_tokens * n_heads * seen * (dim + vdim),
+              elem * kv * n_kv_heads * (2 * dim + vdim) + n_tokens * n_heads * (2 * dim * elem + 8.0 * vdim))
+
+
+def two_map_attention(q, pool, table, table_len, token_seq, positions, out, *, n_tokens, n_heads, n_kv_heads, dim, vdim, scale,
+                      n_splits=1):
+    """Both maps of every head, causal softmax attentions over the pages up to the token's own position, 32-bit
+    multiply-adds.  q [tokens, 2 heads * pad] as differential_prep leaves it.  out (32-bit): [tokens, 2 heads, vdim], or with
+    `n_splits` > 1 the parts [tokens, 2 heads, splits, vdim + 2] that differential_combine joins."""
+    _need(q, "q", (torch.float32, torch.bfloat16))
+    _need(pool, "pool", q.dtype, (None, n_kv_heads, PAGE_SIZE, 2 * dim + vdim))
+    pad = q.shape[1] // (2 * n_heads)
+    if q.shape[0] < n_tokens or pad * 2 * n_heads != q.shape[1] or pad < dim:
+        raise ShapeError("two_map_attention: q does not hold the step's rows")
+    if (out.dtype is not torch.float32 or not out.is_cuda or not out.is_contiguous()
+            or out.numel() < two_map_attention_floats(n_tokens, n_heads, vdim, n_splits)):
+        raise ShapeError("two_map_attention: out is too small")
+    _two_map_work(n_tokens, n_heads, n_kv_heads, dim, vdim, q.element_size(), True)
+    _check(library().bt_two_map_attention(
+        _ptr(q), c_longlong(q.shape[1]), c_int(pad), _ptr(pool), _ptr(table), c_int(table.shape[1]), c_int(table_len),
+        c_int(PAGE_SIZE), _ptr(token_seq), _ptr(positions), _ptr(out), c_int(n_tokens), c_int(n_heads), c_int(n_kv_heads),
+        c_int(dim), c_int(vdim), c_float(scale), c_int(n_splits), c_int(_code(q.dtype)), _stream()))
+
+
+def two_map_attention_tcgen05(q, pool, table, table_len, seq_start, past_len, out, *, n_tokens, n_seqs, max_new, n_heads,
+                              n_kv_heads, dim, vdim, scale):
+    """two_map_attention for runs of many tokens a sequence on the fifth-generation tensor cores (bfloat16; queries padded to
+    64 or 128 channels a map); out [tokens, 2 heads, vdim] 32-bit."""
+    _need(q, "q", torch.bfloat16)
+    _need(pool, "pool", torch.bfloat16, (None, n_kv_heads, PAGE_SIZE, 2 * dim + vdim))
+    pad = q.shape[1] // (2 * n_heads)
+    if q.shape[0] < n_tokens or pad * 2 * n_heads != q.shape[1]:
+        raise ShapeError("two_map_attention_tcgen05: q does not hold the step's rows")
+    if (out.dtype is not torch.float32 or not out.is_cuda or not out.is_contiguous()
+            or out.numel() < two_map_attention_floats(n_tokens, n_heads, vdim, 1)):
+        raise ShapeError("two_map_attention_tcgen05: out is too small")
+    _two_map_work(n_tokens, n_heads, n_kv_heads, dim, vdim, 2, False)
+    _check(library().bt_two_map_attention_tcgen05(
+        _ptr(q), c_longlong(q.shape[0]), c_int(pad), _ptr(pool), c_longlong(pool.shape[0]), _ptr(table), c_int(table.shape[1]),
+        c_int(table_len), _ptr(out), _ptr(kernel_status(q.device)), _ptr(seq_start), _ptr(past_len), c_int(n_seqs),
+        c_int(max_new), c_int(n_heads), c_int(n_kv_heads), c_int(dim), c_int(vdim), c_float(scale), _stream()))
+
+
+def differential_combine(parts, share, gain: float, eps: float, out, *, n_tokens, n_heads, vdim, n_splits=1):
+    """out[t, h] = o / sqrt(mean(o^2) + eps) * gain with o = first map's result - share * the second's, 32-bit; `share` one
+    32-bit number on the device; parts as two_map_attention leaves them; out: [tokens, heads * vdim]."""
+    _need(share, "share", torch.float32, (1,))
+    _need(out, "out", (torch.float32, torch.bfloat16), (None, n_heads * vdim))
+    if (parts.dtype is not torch.float32 or parts.numel() < two_map_attention_floats(n_tokens, n_heads, vdim, n_splits)
+            or out.shape[0] < n_tokens):
+        raise ShapeError("differential_combine: parts or out do not hold the step's rows")
+    _work(0.0, float(n_tokens) * n_heads * vdim * (8.0 * n_splits + out.element_size()))
+    _check(library().bt_differential_combine(_ptr(parts), c_int(n_splits), _ptr(share), c_float(gain), c_float(eps), _ptr(out),
+                                             c_longlong(out.shape[1]), c_int(n_tokens), c_int(n_heads), c_int(vdim),
+                                             c_int(_code(out.dtype)), _stream()))
+
+
+GLA_CHUNK = 64           # runs of more new tokens than this are worked by chunks
+
+
+def gla_chunked_scratch_floats(n_tokens, n_seqs, max_new, n_heads, dim, vdim) -> int:
+    """Floats of scratch: the chunks' states and decays, and the queries carried to their chunk's start."""
+    return n_seqs * -(-max_new // GLA_CHUNK) * n_heads * dim * (vdim + 1) + n_tokens * n_heads * dim
+
+
+def gla_scan_fuses(dim, vdim) -> bool:
+    """Whether the token-by-token kernel holds a whole head of this size in one block (and can norm and gate it)."""
+    return _supports("bt_gla_scan_fuses", dim, vdim)
+
+
+def gla_scan(proj, q_off, k_off, v_off, q_scale: float, dt, log_scale: float, state, slots, seq_start, out, *, n_seqs, n_heads,
+             dim, vdim, max_new, scratch=None, norm=None) -> bool:
+    """Runs S <- diag(exp(log_scale dt)) S + k v^T, o = S^T (q q_scale) over the step's tokens of every sequence; q, k, v are
+    the channels at their offsets in the rows of `proj`, dt [tokens, heads * dim] 32-bit, one number a key channel.
+    state: [slots, heads, dim, vdim] 32-bit, read and written at `slots[seq]`; out: [tokens, heads * vdim] 32-bit.
+
+    Runs of more than GLA_CHUNK tokens with `scratch` (32-bit, gla_chunked_scratch_floats) are worked by chunks, else token
+    by token.  `norm` = (weight [vdim] 32-bit, eps, channel of the output gate in proj's rows, mixed [tokens, heads * vdim]
+    of proj's type): where a block of the token-by-token kernel holds a whole head it leaves
+    o / rms(o) * weight * g sigmoid(g) in `mixed`, writes no `out`, and the call returns True; otherwise False."""
+    _need(proj, "proj", (torch.float32, torch.bfloat16))
+    _need(dt, "dt", torch.float32, (None, n_heads * dim))
+    _need(state, "state", torch.float32, (None, n_heads, dim, vdim))
+    _need(out, "out", torch.float32, (None, n_heads * vdim))
+    if max(q_off, k_off) + n_heads * dim > proj.shape[1] or v_off + n_heads * vdim > proj.shape[1]:
+        raise ShapeError("gla_scan: the channel offsets leave the rows of proj")
+    n_rows = out.shape[0]
+    if dt.shape[0] < n_rows or proj.shape[0] < n_rows:
+        raise ShapeError("gla_scan: proj or dt holds fewer rows than out")
+    _work(4.0 * n_rows * n_heads * dim * vdim, n_rows * n_heads * ((2 * dim + vdim) * proj.element_size() + 4 * dim + 4 * vdim)
+          + 8.0 * n_seqs * n_heads * dim * vdim)
+    common = (_ptr(proj), c_longlong(proj.shape[1]), c_int(q_off), c_int(k_off), c_int(v_off), c_float(q_scale), _ptr(dt),
+              c_float(log_scale), _ptr(state), _ptr(slots), _ptr(seq_start), _ptr(out), c_longlong(out.shape[1]))
+    if max_new > GLA_CHUNK and scratch is not None:
+        need = gla_chunked_scratch_floats(n_rows, n_seqs, max_new, n_heads, dim, vdim)
+        if scratch.dtype != torch.float32 or scratch.numel() < need or not scratch.is_cuda:
+            raise ShapeError(f"gla_scan: runs of {max_new} tokens need {need} floats of scratch")
+        _check(library().bt_gla_chunked(*common, _ptr(scratch), c_int(max_new), c_int(n_seqs), c_int(n_heads), c_int(dim),
+                                        c_int(vdim), c_int(_code(proj.dtype)), _stream()))
+        return False
+    weight = mixed = None
+    eps, g_off = 0.0, 0
+    if norm is not None and gla_scan_fuses(dim, vdim):
+        weight, eps, g_off, mixed = norm
+        _need(weight, "norm weight", torch.float32, (vdim,))
+        _need(mixed, "mixed", proj.dtype, (None, n_heads * vdim))
+        if g_off + n_heads * vdim > proj.shape[1] or mixed.shape[0] < n_rows:
+            raise ShapeError("gla_scan: the gate's channels leave the rows of proj, or mixed is too short")
+    _check(library().bt_gla_scan(*common, c_int(n_seqs), c_int(n_heads), c_int(dim), c_int(vdim), _ptr(weight), c_float(eps),
+                                 c_int(g_off), _ptr(mixed), c_longlong(mixed.shape[1] if mixed is not None else 0),
+                                 c_int(_code(proj.dtype)), _stream()))
+    return weight is not None

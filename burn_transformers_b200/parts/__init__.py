@@ -2,8 +2,10 @@ from .attention import CausalSelfAttention
 from .base import Block, FeedForward, Mixer, Norm, Part, PositionEncoding
 from .block import OutputNormBlock, ParallelBlock, PreNormBlock, SandwichBlock
 from .conv_attention import TalkingConvAttention
+from .differential_attention import DifferentialAttention
 from .embedding import LinearReadout, StreamVectors, TiedReadout, TokenEmbedding
 from .feed_forward import DenseFeedForward, GatedFeedForward, PolyNormFeedForward
+from .gated_linear import GatedLinearAttention
 from .latent_attention import LatentAttention
 from .lightning import LightningAttention, Retention
 from .matrix_memory import MatrixMemory
@@ -21,4 +23,4 @@ __all__ = ["CausalSelfAttention", "Block", "FeedForward", "Mixer", "Norm", "Part
            "LightningAttention", "MatrixMemory", "ParallelBlock", "RoutedFeedForward", "SideBySideMixers",
            "LayerNorm", "RmsNorm", "InterleavedRotary", "LearnedPositions", "NoPositions", "SandwichBlock",
            "TalkingConvAttention", "PolyNormFeedForward", "Retention", "SelectiveScan", "HalfSplitRotary", "OutputNormBlock",
-           "SigmoidAttention", "TokenShift", "MinGru"]
+           "SigmoidAttention", "TokenShift", "MinGru", "DifferentialAttention", "GatedLinearAttention"]

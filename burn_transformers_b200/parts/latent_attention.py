@@ -32,7 +32,8 @@ class LatentAttention(Mixer):
     of latents.  A layer built with `owns_latent=False` has no W_dkv; the model's run order gives it another layer's
     cache entry, whose rows it reads with its own W_uk, W_uv, queries and everything else.
 
-    By argument: `gate=False` leaves the output gate out; `window` = W lets position i see j with 0 <= i - j < W only;
+    By argument: `gate=False` leaves the output gate out, `gate="head"` makes it one number a head, sigmoid(W_g h)_i, with
+    W_g of `heads` rows (followed by zero rows up to `gate_width`, a multiple of 8); `window` = W lets position i see j with 0 <= i - j < W only;
     `q_rank` = r sends the queries through a latent of their own, c_q = (W_dq h) / rms(W_dq h) * q_norm, q = W_uq c_q
     (then `in.weight` opens with W_dq's r rows in W_q's place, and the part has `q_norm.weight` [r] and `uq.weight`
     [heads * (dim + rot_dim), r]).  A windowed layer keeps every position in its pages all the same: the kernels skip
@@ -55,7 +56,7 @@ class LatentAttention(Mixer):
 
     def __init__(self, width: int, n_heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float, eps: float,
                  positions, *, owns_latent: bool = True, sink: bool = True, init_std: float = 0.02,
-                 out_init_std: float | None = None, gate: bool = True, window: int | None = None,
+                 out_init_std: float | None = None, gate: bool | str = True, window: int | None = None,
                  q_rank: int | None = None):
         if min(width, n_heads, dim, vdim, kv_rank) <= 0 or rot_dim < 0:
             raise ShapeError("latent attention: sizes must be positive")
@@ -65,13 +66,18 @@ class LatentAttention(Mixer):
             raise ShapeError("latent attention: needs a rotating position encoding over at most rot_dim channels")
         self.width, self.n_heads, self.dim, self.rot_dim, self.vdim, self.kv_rank = width, n_heads, dim, rot_dim, vdim, kv_rank
         self.scale, self.eps, self.positions = float(scale), float(eps), positions
+        if getattr(positions, "size", 1.0) != 1.0:
+            raise ShapeError("latent attention: its kernels do not scale sine and cosine")
+        if gate not in (True, False, "head"):
+            raise ShapeError(f"latent attention: an output gate is True, False or \"head\", not {gate!r}")
         if (window is not None and window <= 0) or (q_rank is not None and q_rank <= 0):
             raise ShapeError("latent attention: a window and a query latent are positive")
-        self.owns_latent, self.has_sink, self.has_gate = owns_latent, sink, gate
+        self.owns_latent, self.has_sink, self.has_gate = owns_latent, sink, bool(gate)
+        self.gate_per_head = gate == "head"
         self.window, self.q_rank = window, q_rank
         self.q_width = n_heads * (dim + rot_dim)
         self.mixed_width = n_heads * vdim
-        self.gate_width = self.mixed_width if gate else 0
+        self.gate_width = -(-n_heads // 8) * 8 if self.gate_per_head else self.mixed_width if gate else 0
         self.latent_width = kv_rank + rot_dim
         self.q_in_width = self.q_width if q_rank is None else q_rank      # what the first product gives of the queries
         self.in_width = self.q_in_width + self.gate_width + (self.latent_width if owns_latent else 0)
@@ -170,7 +176,8 @@ class LatentAttention(Mixer):
             mixed = ctx.ws.take((n, self.mixed_width), dtype)
             kernels.latent_decode_finish(self.uv_heads, mixed, n_tokens=n, n_splits=splits, scratch=scratch,
                                          mixed_latent=mixed_latent,
-                                         gate=proj[:, gate_off:latent_off] if self.has_gate else None)
+                                         gate=proj[:, gate_off:gate_off + (heads if self.gate_per_head else self.mixed_width)]
+                                         if self.has_gate else None)
             linear(ctx, mixed, self.t_out_weight, None, residual, m=n, residual=None if store else residual, w_is_nk=True)
             ctx.ws.release(mark)
             return
@@ -179,7 +186,11 @@ class LatentAttention(Mixer):
                                   ctx.positions, ctx.token_seq, freq, self.positions.dims, table, group.table_len, pool,
                                   n, rank, rot)
         q_heads = queries[:, :self.q_width].view(n, heads, self.dim + rot)
-        gate = proj[:, gate_off:latent_off].view(n, heads, self.vdim) if self.has_gate else None
+        gate = None
+        if self.gate_per_head:
+            gate = proj[:, gate_off:gate_off + heads].unsqueeze(2).expand(n, heads, self.vdim)
+        elif self.has_gate:
+            gate = proj[:, gate_off:latent_off].view(n, heads, self.vdim)
         if dtype == torch.bfloat16 and ctx.fresh and not ctx.is_decode and ctx.max_new >= self.plain_from:
             # fresh prompts: the step's own latent rows, keys and values per head, ordinary attention
             rows = ctx.ws.take((n, dk), dtype)

@@ -67,20 +67,21 @@ def linear(ctx, a, w, bias, out, *, m, w_is_nk=False, activation=None, residual=
         return
     if w.dtype == torch.bfloat16 and m <= 64:
         fuse = lazy and m <= 16 and a.norm.fusable
+        rms = fuse and a.norm.fused_kind == "rmsnorm"
         if w_is_nk and n >= 8192 and kernels.linear_stream_supports(m, n, k, fuse):
             # a wide [N, K] table (the readout): long weight rows, streamed straight into registers
             if lazy and not fuse:
                 a, lazy = a.materialize(ctx), False
             norm = (a.x32, a.norm.t_weight, a.norm.t_bias if a.norm.has_bias else None, a.norm.eps, a.rows) if lazy else None
             kernels.linear_stream(None if lazy else a, w, bias, out, m=m, activation=activation, residual=residual,
-                                  norm=norm)
+                                  norm=norm, rms=rms)
             return
         if kernels.linear_skinny_supports(m, n, k, w_is_nk, fuse):
             if lazy and not fuse:
                 a, lazy = a.materialize(ctx), False
             norm = (a.x32, a.norm.t_weight, a.norm.t_bias if a.norm.has_bias else None, a.norm.eps, a.rows) if lazy else None
             kernels.linear_skinny(None if lazy else a, w, bias, out, m=m, w_is_nk=w_is_nk, activation=activation,
-                                  residual=residual, norm=norm)
+                                  residual=residual, norm=norm, rms=rms)
             return
     if lazy:
         a = a.materialize(ctx)

@@ -61,8 +61,13 @@ class RmsNorm(Norm):
             tensors = {name: t.to(torch.float32).reshape(1).expand(self.width).contiguous() for name, t in tensors.items()}
         super().bind(tensors)
 
+    fusable = True      # (as LayerNorm: the products for few rows norm on the way in)
+    fused_kind = "rmsnorm"
+
     def forward(self, ctx, x32, out_dtype, rows=None, n_rows=None, lazy=False):
         n = n_rows if n_rows is not None else ctx.n_tokens
+        if lazy and out_dtype == torch.bfloat16 and n <= 16:
+            return LazyNorm(self, x32, rows, n)
         return self.apply(ctx, x32, out_dtype, rows, n)
 
     def apply(self, ctx, x32, out_dtype, rows, n):

@@ -37,10 +37,16 @@ class InterleavedRotary(PositionEncoding):
 
     `stretch` = (factor, low, high, original) slows the long waves down: with the wavelength l = 2 pi / f of a
     frequency f, f stays where l < original / high, becomes f / factor where l > original / low, and in between is
-    (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
+    (1 - s) f / factor + s f with s = (original / l - low) / (high - low).
+
+    `yarn` = (factor, original, fast, slow) does so by the pair's index instead: with d(t) = dims ln(original / (2 pi t)) /
+    (2 ln base) the index of the pair that turns t times within `original` positions, lo = max(floor d(fast), 0) and hi =
+    min(ceil d(slow), dims - 1), pair i keeps the share 1 - r of f and takes the share r of f / factor, r = (i - lo) /
+    max(hi - lo, 0.001) clamped to [0, 1]; sine and cosine are multiplied by `size` = 0.1 ln(factor) + 1 (1 without it)."""
     rotates = True
 
-    def __init__(self, dims: int, base: float, stretch: tuple[float, float, float, float] | None = None):
+    def __init__(self, dims: int, base: float, stretch: tuple[float, float, float, float] | None = None,
+                 yarn: tuple[float, float, float, float] | None = None):
         if dims < 0 or dims % 2:
             raise ValueError(f"a rotation takes an even number of channels, not {dims}")
         self.dims, self.base = int(dims), float(base)
@@ -48,11 +54,26 @@ class InterleavedRotary(PositionEncoding):
         if self.stretch is not None and (len(self.stretch) != 4 or self.stretch[0] <= 0 or self.stretch[3] <= 0
                                          or self.stretch[2] <= self.stretch[1]):
             raise ValueError(f"a stretch is (factor > 0, low, high > low, original > 0), not {stretch}")
+        self.yarn = None if yarn is None else tuple(float(v) for v in yarn)
+        if self.yarn is not None and (stretch is not None or len(self.yarn) != 4 or min(self.yarn) <= 0 or base <= 1):
+            raise ValueError(f"yarn is (factor, original, fast, slow), all positive, over a base above 1 and without a "
+                             f"stretch, not {yarn}")
+        self.size = 1.0 if self.yarn is None else 0.1 * math.log(self.yarn[0]) + 1.0
         self._freq: dict = {}
 
     def frequencies(self) -> list[float]:
         """The dims / 2 frequencies, in 64-bit."""
         values = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if self.yarn is not None and self.dims:
+            factor, original, fast, slow = self.yarn
+
+            def pair_that_turns(times):
+                return self.dims * math.log(original / (2.0 * math.pi * times)) / (2.0 * math.log(self.base))
+
+            lo = max(math.floor(pair_that_turns(fast)), 0)
+            hi = min(math.ceil(pair_that_turns(slow)), self.dims - 1)
+            shares = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(len(values))]
+            return [f / factor * r + f * (1.0 - r) for f, r in zip(values, shares)]
         if self.stretch is None:
             return values
         factor, low, high, original = self.stretch
@@ -81,6 +102,8 @@ class InterleavedRotary(PositionEncoding):
 
     def rotate_vectors(self, ctx, src, dst) -> None:
         """dst[t, v, :] = src[t, v, :] turned by the position of token t (views [tokens, vectors, length])."""
+        if self.size != 1.0:
+            raise NotImplementedError("this kernel does not scale sine and cosine")
         kernels.rotary_interleaved(src, dst, ctx.positions, self.inv_freq(src.device), n_tokens=ctx.n_tokens,
                                    dims=self.dims)
 
@@ -98,6 +121,8 @@ class HalfSplitRotary(InterleavedRotary):
 
     def rotate_rows(self, ctx, src, dst, *, n_vecs: int, length: int, scaled_from=None, scale: float = 1.0,
                     tail: int = 0) -> None:
+        if self.size != 1.0:
+            raise NotImplementedError("this kernel does not scale sine and cosine")
         kernels.rotary_half(src, dst, ctx.positions, self.inv_freq(src.device), n_tokens=ctx.n_tokens, n_vecs=n_vecs,
                             length=length, dims=self.dims, scaled_from=scaled_from, scale=scale, tail=tail)
 
