@@ -310,7 +310,7 @@ def linear_mid(a, w, bias, out, *, m, activation=None, residual=None, split=0):
     _linear_work(m, n, k, a, w, out)
     _check(library().bt_linear_mid(_ptr(a), _ptr(w), _ptr(bias), _ptr(residual), _ptr(out), _ptr(kernel_status(a.device)),
                                    c_int(m), c_int(n), c_int(k), c_int(ACTIVATIONS[activation]),
-                                   c_int(1 if out.dtype == torch.float32 else 0), c_int(split), c_int(1 if rms else 0), _stream()))
+                                   c_int(1 if out.dtype == torch.float32 else 0), c_int(split), _stream()))
 
 
 def linear_mid_supports(m, n, k) -> bool:
