@@ -1,7 +1,7 @@
 """Decode and prefill throughput of GPT-2 (random weights, synthetic tokens) on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--points all|small] [--profile]
-    python bench.py --arch sovozen|gokezen|rakarax|bosalix|visadra [--sizes small,medium]
+    python bench.py --arch sovozen|gokezen|rakarax|bosalix|visadra|zatinex [--sizes small,medium]
 
 A step is one decode step of a batch of 8 sequences of GPT-2 small.  The run prints one JSON line: `value` is decoded
 tokens per second, timed on the device with CUDA events over exactly K steps; `e2e` is the same through the public
@@ -461,15 +461,39 @@ def visadra(size: str) -> dict:
             "logit_scale": 1.0, "layers": layers}
 
 
+def zatinex(size: str) -> dict:
+    """A Zatinex with as many layers and the width of GPT-2 `size`: in turn a latent attention with a latent of its own
+    (256 or 512 + 32 or 64 rotated, queries through a latent of half the width), a differential attention (half of GPT-2's
+    heads with two maps of 64 channels and values of 128 each, a key head for every two query heads, a convolution of 4
+    taps, a scaled rotation), a gated linear attention (GPT-2's heads, 64 x 64 states, decays through 16 numbers) and a
+    latent attention that reads the first one's latent; gated feed-forwards of the same weight count as GPT-2's."""
+    n_layer, width, heads = {"small": (12, 768, 12), "medium": (24, 1024, 16)}[size]
+    rank, rot, ff = {"small": (256, 32, 2048), "medium": (512, 64, 2816)}[size]
+    dim = 64
+    mlp = {"kind": "dense", "ff": ff}
+    latent = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": dim, "kv_rank": rank, "q_rank": width // 2,
+              "scale": (dim + rot) ** -0.5, "rot": {"dims": rot, "base": 10000.0}}
+    attention = {"heads": heads // 2, "kv_heads": heads // 4, "dim": dim, "vdim": 2 * dim, "conv": 4, "scale": dim ** -0.5,
+                 "diff": 0.5, "rot": {"dims": dim // 2, "base": 10000.0,
+                                      "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    gla = {"heads": heads, "dim": dim, "vdim": dim, "tau": 16.0, "decay_rank": 16}
+    layers = []
+    for i in range(n_layer):
+        kind, mixer = (("latent_attention", latent), ("attention", attention), ("gla", gla),
+                       ("latent_attention", dict(latent, kv_from=i - 3)))[i % 4]
+        layers.append({"type": kind, "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Zatinex", "vocab": 50257, "width": width, "norm": {"eps": 1e-5}, "layers": layers}
+
+
 ARCH_PAIRS = {"sovozen": (sovozen, "gpt2", gpt2), "gokezen": (gokezen, "sovozen", sovozen),
               "rakarax": (rakarax, "gokezen", gokezen), "bosalix": (bosalix, "gokezen", gokezen),
-              "visadra": (visadra, "bosalix", bosalix)}
+              "visadra": (visadra, "bosalix", bosalix), "zatinex": (zatinex, "sovozen", sovozen)}
 
 
 def run_arch_compare(args):
-    """--arch sovozen | gokezen | rakarax | bosalix | visadra: prefill and decode throughput of that design beside the library's
+    """--arch sovozen | gokezen | rakarax | bosalix | visadra | zatinex: prefill and decode throughput of that design beside the library's
     closest other model at the same width and depth (GPT-2 for Sovozen, Sovozen for Gokezen, Gokezen for Rakarax and for
-    Bosalix, Bosalix for Visadra; random weights, bfloat16), and where each
+    Bosalix, Bosalix for Visadra, Sovozen for Zatinex; random weights, bfloat16), and where each
     spends a prefill and a decode step, kernel by kernel, against the measured peaks.  One JSON line; the default
     workload of this file is untouched."""
     import numpy as np
@@ -690,8 +714,8 @@ def main() -> int:
     parser.add_argument("--profile", action="store_true",
                         help="print where a prefill and a decode step spend their time, kernel by kernel, instead")
     parser.add_argument("--model", choices=["small", "medium", "xl"], default="small", help="the model --profile looks at")
-    parser.add_argument("--arch", choices=["gpt2", "sovozen", "gokezen", "rakarax", "bosalix", "visadra"], default="gpt2",
-                        help="sovozen, gokezen, rakarax, bosalix, visadra: measure that design beside the closest other model of equal width and "
+    parser.add_argument("--arch", choices=["gpt2", "sovozen", "gokezen", "rakarax", "bosalix", "visadra", "zatinex"], default="gpt2",
+                        help="sovozen, gokezen, rakarax, bosalix, visadra, zatinex: measure that design beside the closest other model of equal width and "
                              "depth instead (see --sizes)")
     parser.add_argument("--sizes", default="small,medium", help="with an --arch other than gpt2: which widths (small, medium)")
     args = parser.parse_args()
