@@ -222,7 +222,8 @@ int bt_moe_combine(const float* part, const int* place, float* stream_rows, long
 int bt_differential_prep(const void* proj, long long row_stride, const float* conv, float* state, const int* slots,
                          const int* seq_start, const int* token_seq, const int* positions, const float* q_weight,
                          const float* k_weight, float eps, const float* inv_freq, int rot_dims, float rot_size, int taps,
-                         const int* table, int table_stride, int table_len, int page_size, void* pool, void* q_out, int q_pad,
+                         const int* table, int table_stride, int table_len, int page_size, void* pool, long long pool_pages,
+                         void* q_out, int q_pad,
                          int n_tokens, int n_seqs, int max_new, int n_heads, int n_kv_heads, int dim, int vdim, int dtype,
                          cudaStream_t stream);
 int bt_two_map_attention(const void* q, long long q_row_stride, int q_pad, const void* pool, const int* table, int table_stride,

@@ -88,10 +88,22 @@ __global__ void __launch_bounds__(128) differential_prep_kernel(DiffPrepArgs p) 
   const T* src = reinterpret_cast<const T*>(p.proj) + ch0;
   const bool word = p.pairs_ok != 0;
   const int dkv = 2 * p.dim + p.vdim;
-  const int t_end = min(p.n_tokens, (int)(blockIdx.x + 1) * p.run);
-  for (int t = blockIdx.x * p.run; t < t_end; ++t) {
-    const int seq = p.token_seq[t], r = t - p.seq_start[seq], pos = p.positions[t];
-    float* kept = p.state + (long long)p.slots[seq] * (taps - 1) * channels + ch0;
+  const int t_first = blockIdx.x * p.run, t_end = min(p.n_tokens, t_first + p.run);
+  // where the run's tokens lie: lane i looks up token i, so that the look-ups of a run wait for one another once
+  int at_r = 0, at_pos = 0, at_slot = 0, at_row = 0;
+  if (t_first + lane < t_end) {
+    const int t = t_first + lane, seq = p.token_seq[t];
+    at_pos = p.positions[t];
+    at_r = t - p.seq_start[seq];
+    at_slot = p.slots[seq];
+    const int lp = at_pos / p.page_size;
+    at_row = p.table[(long long)seq * p.table_stride + (lp % p.table_len)] * p.n_kv_heads * p.page_size + at_pos - lp * p.page_size;
+  }
+  for (int t = t_first; t < t_end; ++t) {
+    const int r = __shfl_sync(0xffffffffu, at_r, t - t_first), pos = __shfl_sync(0xffffffffu, at_pos, t - t_first);
+    const int slot = __shfl_sync(0xffffffffu, at_slot, t - t_first);
+    const long long pool_row = __shfl_sync(0xffffffffu, at_row, t - t_first);
+    float* kept = p.state + (long long)slot * (taps - 1) * channels + ch0;
     float2 y[PJ];
     float ss = 0.f;
 #pragma unroll
@@ -141,10 +153,8 @@ __global__ void __launch_bounds__(128) differential_prep_kernel(DiffPrepArgs p) 
     if (is_q) {
       dst = reinterpret_cast<T*>(p.q_out) + (long long)t * q_units * p.q_pad + (long long)unit * p.q_pad;
     } else {
-      const int lp = pos / p.page_size;
-      const long long page = p.table[(long long)seq * p.table_stride + (lp % p.table_len)];
       const int g = is_k ? (unit - q_units) >> 1 : unit - q_units - k_units;
-      dst = reinterpret_cast<T*>(p.pool) + ((page * p.n_kv_heads + g) * p.page_size + (pos - lp * p.page_size)) * dkv +
+      dst = reinterpret_cast<T*>(p.pool) + (pool_row + (long long)g * p.page_size) * dkv +
             (is_k ? ((unit - q_units) & 1) * p.dim : 2 * p.dim);
     }
     const float inv = weight != nullptr ? 1.f / sqrtf(warp_sum(ss) / (float)len + p.eps) : 1.f;
@@ -556,11 +566,12 @@ extern "C" int bt_differential_prep(const void* proj, long long row_stride, cons
                                     const int* seq_start, const int* token_seq, const int* positions, const float* q_weight,
                                     const float* k_weight, float eps, const float* inv_freq, int rot_dims, float rot_size,
                                     int taps, const int* table, int table_stride, int table_len, int page_size, void* pool,
-                                    void* q_out, int q_pad, int n_tokens, int n_seqs, int max_new, int n_heads, int n_kv_heads,
+                                    long long pool_pages, void* q_out, int q_pad, int n_tokens, int n_seqs, int max_new, int n_heads, int n_kv_heads,
                                     int dim, int vdim, int dtype, cudaStream_t stream) {
   using namespace bt;
+  // (a pool's rows are counted in 32 bits)
   BT_CHECK(n_tokens >= 0 && n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0 && dim > 0 && dim <= 256 && vdim > 0 &&
-               vdim <= 256 && rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && taps >= 1 && taps <= DA_MAX_TAPS &&
+               vdim <= 256 && pool_pages > 0 && pool_pages * n_kv_heads * page_size < (1ll << 31) && rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && taps >= 1 && taps <= DA_MAX_TAPS &&
                q_pad >= dim,
            "differential_prep: bad sizes heads=%d kv_heads=%d dim=%d vdim=%d (up to 256) rot_dims=%d taps=%d (up to %d)", n_heads,
            n_kv_heads, dim, vdim, rot_dims, taps, DA_MAX_TAPS);

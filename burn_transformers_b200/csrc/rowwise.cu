@@ -72,6 +72,75 @@ rmsnorm_warp_kernel(const TIn* __restrict__ x, long long x_row_stride, const flo
   }
 }
 
+__device__ __forceinline__ void store_four(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_four(__nv_bfloat16* p, const float4& v) {
+  uint2 o;
+  *reinterpret_cast<__nv_bfloat162*>(&o.x) = __floats2bfloat162_rn(v.x, v.y);
+  *reinterpret_cast<__nv_bfloat162*>(&o.y) = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = o;
+}
+__device__ __forceinline__ float square_sum(const float4& v, float s) {
+  return fmaf(v.w, v.w, fmaf(v.z, v.z, fmaf(v.y, v.y, fmaf(v.x, v.x, s))));
+}
+__device__ __forceinline__ void add_four(float4& v, const float4& a) { v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w; }
+__device__ __forceinline__ float4 load_four(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load_four(const __nv_bfloat16* p) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// The same for runs of whole 4-channel pieces, at most 4 * LPR * NV channels: LPR adjacent lanes a run, every operand read
+// once in 16- or 8-byte pieces; the weights (which no kernel of a step writes) and the gates are asked for before the sum.
+template <typename TIn, typename TGate, typename TOut, int LPR, int NV>
+__global__ void __launch_bounds__(128)
+rmsnorm_pieces_kernel(const TIn* __restrict__ x, long long x_row_stride, const float* __restrict__ weight,
+                      const TGate* __restrict__ gate, long long gate_row_stride, TOut* __restrict__ out,
+                      long long out_row_stride, int width, int groups, long long items, float eps, int gate_rule) {
+  pdl_trigger();
+  const long long item = (long long)blockIdx.x * (128 / LPR) + threadIdx.x / LPR;
+  const int lane = threadIdx.x % LPR;
+  const bool live = item < items;
+  const long long r = live ? item / groups : 0;
+  const int first = live ? (int)(item - r * groups) * width : 0;
+  float4 w[NV], v[NV], g[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = 4 * (lane + LPR * i);
+    w[i] = v[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (live && c < width) w[i] = load_four(weight + first + c);
+  }
+  pdl_wait();
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = 4 * (lane + LPR * i);
+    if (live && c < width) {
+      v[i] = load_four(x + r * x_row_stride + first + c);
+      if (gate) g[i] = load_four(gate + r * gate_row_stride + first + c);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) ss = square_sum(v[i], ss);
+#pragma unroll
+  for (int o = LPR >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = 1.f / sqrtf(ss / (float)width + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = 4 * (lane + LPR * i);
+    if (!live || c >= width) continue;
+    float4 y = make_float4(v[i].x * inv * w[i].x, v[i].y * inv * w[i].y, v[i].z * inv * w[i].z, v[i].w * inv * w[i].w);
+    if (gate) {
+      y.x *= gate_value(g[i].x, gate_rule);
+      y.y *= gate_value(g[i].y, gate_rule);
+      y.z *= gate_value(g[i].z, gate_rule);
+      y.w *= gate_value(g[i].w, gate_rule);
+    }
+    store_four(out + r * out_row_stride + first + c, y);
+  }
+}
+
 // dst[t, v, :] = src[t, v, :] with the pairs (2i, 2i+1), i < dims/2, turned by positions[t] * inv_freq[i]; the
 // channels from `dims` to `len` are copied.  src and dst may be the same memory.
 template <typename T>
@@ -180,6 +249,28 @@ static int launch_rmsnorm(const TIn* x, long long xs, const float* w, const TGat
                           cudaStream_t stream) {
   width /= groups;
   const long long items = (long long)n_rows * groups;
+  auto lies = [](const void* p, long long stride, size_t elem) {
+    return stride % 4 == 0 && (unsigned long long)p % (4 * elem) == 0;
+  };
+  if (width <= 1024 && width % 4 == 0 && lies(x, xs, sizeof(TIn)) && lies(out, os, out_dtype == kF32 ? 4 : 2) && lies(w, 0, 4) &&
+      (gate == nullptr || lies(gate, gs, sizeof(TGate)))) {
+#define BT_RP_KIND(TOUT, LPR, NV)                                                                                         \
+  BT_PDL_OK("rmsnorm", launch_pdl(rmsnorm_pieces_kernel<TIn, TGate, TOUT, LPR, NV>,                                       \
+                                  dim3((unsigned)((items + 128 / LPR - 1) / (128 / LPR))), dim3(128), 0, stream, 1, x, xs, w, \
+                                  gate, gs, (TOUT*)out, os, width, groups, items, eps, gate_rule))
+#define BT_RP(LPR, NV)                                                                                                    \
+  do {                                                                                                                    \
+    if (out_dtype == kF32) BT_RP_KIND(float, LPR, NV); else BT_RP_KIND(__nv_bfloat16, LPR, NV);                           \
+  } while (0)
+    if (width <= 64) BT_RP(16, 1);
+    else if (width <= 128) BT_RP(32, 1);
+    else if (width <= 512) BT_RP(32, 4);
+    else if (width <= 768) BT_RP(32, 6);
+    else BT_RP(32, 8);
+#undef BT_RP
+#undef BT_RP_KIND
+    return 0;
+  }
   if (width <= 1024) {
     const dim3 wgrid((unsigned)((items + 3) / 4));
 #define BT_RW(TOUT, NV)                                                                                              \
@@ -362,17 +453,6 @@ __global__ void __launch_bounds__(128) rmsnorm_add_kernel(NormAddArgs p) {
     next_out[r * p.width + c] = from_float<TOut>(dst[c] * inv2 * p.next_weight[c]);
 }
 
-__device__ __forceinline__ void store_four(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void store_four(__nv_bfloat16* p, const float4& v) {
-  uint2 o;
-  *reinterpret_cast<__nv_bfloat162*>(&o.x) = __floats2bfloat162_rn(v.x, v.y);
-  *reinterpret_cast<__nv_bfloat162*>(&o.y) = __floats2bfloat162_rn(v.z, v.w);
-  *reinterpret_cast<uint2*>(p) = o;
-}
-__device__ __forceinline__ float square_sum(const float4& v, float s) {
-  return fmaf(v.w, v.w, fmaf(v.z, v.z, fmaf(v.y, v.y, fmaf(v.x, v.x, s))));
-}
-__device__ __forceinline__ void add_four(float4& v, const float4& a) { v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w; }
 
 // The same for rows of whole 16-byte pieces, at most NV of them a thread: the row stays in registers, every operand is
 // read once, and all reads that do not wait for the sum are asked for before it.

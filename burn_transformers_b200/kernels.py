@@ -1669,8 +1669,8 @@ def differential_prep(proj, conv, state, slots, seq_start, token_seq, positions,
     _check(library().bt_differential_prep(
         _ptr(proj), c_longlong(proj.shape[1]), _ptr(conv), _ptr(state), _ptr(slots), _ptr(seq_start), _ptr(token_seq),
         _ptr(positions), _ptr(q_weight), _ptr(k_weight), c_float(eps), _ptr(inv_freq), c_int(rot_dims), c_float(rot_size),
-        c_int(taps), _ptr(table), c_int(table.shape[1]), c_int(table_len), c_int(PAGE_SIZE), _ptr(pool), _ptr(q_out), c_int(pad),
-        c_int(n_tokens), c_int(n_seqs), c_int(max_new), c_int(n_heads), c_int(n_kv_heads), c_int(dim), c_int(vdim),
+        c_int(taps), _ptr(table), c_int(table.shape[1]), c_int(table_len), c_int(PAGE_SIZE), _ptr(pool),
+        c_longlong(pool.shape[0]), _ptr(q_out), c_int(pad), c_int(n_tokens), c_int(n_seqs), c_int(max_new), c_int(n_heads), c_int(n_kv_heads), c_int(dim), c_int(vdim),
         c_int(_code(proj.dtype)), _stream()))
 
 
