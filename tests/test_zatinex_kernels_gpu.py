@@ -180,7 +180,7 @@ def test_convolution_norm_rotation_and_filing(dtype, tol, heads, groups, dim, vd
         q_out = torch.full((n + 1, 2 * heads * pad), 9.0, dtype=dtype, device=DEV)
         token_seq = ints(np.repeat(range(3), news))
         place = ints(np.concatenate([np.arange(d, d + c) for d, c in zip(done, news)]))
-        kernels.differential_prep(proj, dev(conv.T), state if taps > 1 else state[:, :0], ints(slots), starts(news), token_seq, place,
+        kernels.differential_prep(proj, dev(np.ascontiguousarray(conv.T)), state if taps > 1 else state[:, :0], ints(slots), starts(news), token_seq, place,
                                   dev(gains[0]) if normed else None, dev(gains[1]) if normed else None, 1e-4,
                                   positions.inv_freq(DEV), rot, positions.size, t.pages, t.width, t.pool, q_out[:n], n_tokens=n,
                                   n_seqs=3, max_new=max(news), n_heads=heads, n_kv_heads=groups, dim=dim, vdim=vdim)
