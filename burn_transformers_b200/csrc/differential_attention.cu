@@ -33,7 +33,7 @@ struct DiffPrepArgs {
   int n_tokens, n_heads, n_kv_heads, dim, vdim, q_pad;
   int run;                         // consecutive tokens a warp takes
   int shift_state;                 // every sequence brings one token: the kernel moves the state on itself
-  int pairs_ok;                    // two adjacent channels may be read as one word
+  int pairs_ok;                    // two adjacent channels may be read and written as one word
 };
 
 template <typename T>
@@ -49,113 +49,141 @@ __device__ __forceinline__ float2 da_pair<__nv_bfloat16>(const __nv_bfloat16* p,
   return make_float2(to_float(p[0]), second ? to_float(p[1]) : 0.f);
 }
 
-// A warp takes one unit (a map of a query or key head, or a value head) of `run` consecutive tokens; a lane owns PJ channel
-// pairs of it, 64 channels apart, with their taps in registers where TAPS says how many there are (0: any number).
+__device__ __forceinline__ void da_store_pair(float* p, float a, float b, bool second, bool word) {
+  if (word && second) { *reinterpret_cast<float2*>(p) = make_float2(a, b); return; }
+  p[0] = a;
+  if (second) p[1] = b;
+}
+__device__ __forceinline__ void da_store_pair(__nv_bfloat16* p, float a, float b, bool second, bool word) {
+  if (word && second) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); return; }
+  p[0] = __float2bfloat16_rn(a);
+  if (second) p[1] = __float2bfloat16_rn(b);
+}
+
+constexpr int DA_PREP_WARPS = 8;
+constexpr int DA_RUN = 8;          // consecutive tokens a warp takes at most
+
+// A warp takes one unit (a map of a query or key head, or 64 PJ channels of a value head) of `run` consecutive tokens; a lane
+// owns PJ channel pairs of it, 64 channels apart.  Where TAPS says how many taps there are (0: any number), taps and the
+// last TAPS - 1 inputs stay in registers, so every input is read once a run.  The block's warps take the same tokens: sines
+// and cosines of the run are formed once for all of them.
 template <typename T, int TAPS, int PJ>
-__global__ void __launch_bounds__(128) differential_prep_kernel(DiffPrepArgs p) {
+__global__ void __launch_bounds__(DA_PREP_WARPS * 32) differential_prep_kernel(DiffPrepArgs p) {
+  extern __shared__ float2 turn[];       // [run][rot_dims / 2]: (cosine, sine) times rot_size
   const int lane = threadIdx.x & 31;
-  const int q_units = 2 * p.n_heads, k_units = 2 * p.n_kv_heads, units = q_units + k_units + p.n_kv_heads;
-  const int unit = blockIdx.y * 4 + (threadIdx.x >> 5);
+  const int v_pieces = (p.vdim + 64 * PJ - 1) / (64 * PJ);
+  const int q_units = 2 * p.n_heads, k_units = 2 * p.n_kv_heads, units = q_units + k_units + p.n_kv_heads * v_pieces;
+  const int unit = blockIdx.y * DA_PREP_WARPS + (threadIdx.x >> 5);
   const int taps = TAPS > 0 ? TAPS : p.taps;
-  pdl_trigger();
-  if (unit >= units) return;
-  const bool is_q = unit < q_units, is_k = !is_q && unit < q_units + k_units;
-  const int len = is_q || is_k ? p.dim : p.vdim;
-  const int ch0 = is_q || is_k ? unit * p.dim : (q_units + k_units) * p.dim + (unit - q_units - k_units) * p.vdim;
   const int channels = (q_units + k_units) * p.dim + p.n_kv_heads * p.vdim;
+  const bool works = unit < units, is_q = unit < q_units, is_k = !is_q && unit < q_units + k_units;
+  const bool is_v = works && !is_q && !is_k;
+  const int v_unit = unit - q_units - k_units, v_head = v_unit / v_pieces, v_first = (v_unit - v_head * v_pieces) * 64 * PJ;
+  const int len = is_v ? min(64 * PJ, p.vdim - v_first) : p.dim;
+  const int ch0 = is_v ? (q_units + k_units) * p.dim + v_head * p.vdim + v_first : unit * p.dim;
+  const float* weight = is_q ? p.q_weight : (is_k ? p.k_weight : nullptr);
+  pdl_trigger();
   float2 w[TAPS > 0 ? TAPS : 1][PJ];
   float2 gain[PJ];
-  float freq[PJ];
-  const float* weight = is_q ? p.q_weight : (is_k ? p.k_weight : nullptr);
+  if (works) {
 #pragma unroll
-  for (int j = 0; j < PJ; ++j) {
-    const int c = 2 * (lane + 32 * j);
-    gain[j] = make_float2(1.f, 1.f);
-    freq[j] = 0.f;
-    if (c < len) {
-      if (weight != nullptr) gain[j] = make_float2(weight[c], c + 1 < len ? weight[c + 1] : 0.f);
-      if ((is_q || is_k) && c < p.rot_dims) freq[j] = p.inv_freq[c >> 1];
-    }
-    if (TAPS > 0) {
+    for (int j = 0; j < PJ; ++j) {
+      const int c = 2 * (lane + 32 * j);
+      gain[j] = make_float2(1.f, 1.f);
+      if (weight != nullptr && c < len) gain[j] = make_float2(weight[c], c + 1 < len ? weight[c + 1] : 0.f);
+      if (TAPS > 0) {
 #pragma unroll
-      for (int k = 0; k < TAPS; ++k)
-        w[k][j] = c < len ? make_float2(p.conv[(long long)k * channels + ch0 + c],
-                                        c + 1 < len ? p.conv[(long long)k * channels + ch0 + c + 1] : 0.f)
-                          : make_float2(0.f, 0.f);
+        for (int k = 0; k < TAPS; ++k)
+          w[k][j] = c < len ? make_float2(p.conv[(long long)k * channels + ch0 + c],
+                                          c + 1 < len ? p.conv[(long long)k * channels + ch0 + c + 1] : 0.f)
+                            : make_float2(0.f, 0.f);
+      }
     }
   }
   pdl_wait();
+  const int t_first = blockIdx.x * p.run, t_end = min(p.n_tokens, t_first + p.run), half = p.rot_dims >> 1;
+  for (int i = threadIdx.x; i < (t_end - t_first) * half; i += DA_PREP_WARPS * 32) {
+    const int t = i / half, pair = i - t * half;
+    float sn, cs;
+    sincosf((float)p.positions[t_first + t] * p.inv_freq[pair], &sn, &cs);
+    turn[i] = make_float2(cs * p.rot_size, sn * p.rot_size);
+  }
+  // where the run's tokens lie: lane i looks up token i, so that the look-ups of a run wait for one another once
+  int at_r = 0, at_slot = 0, at_row = 0;
+  if (t_first + lane < t_end) {
+    const int t = t_first + lane, seq = p.token_seq[t], pos = p.positions[t];
+    at_r = t - p.seq_start[seq];
+    at_slot = p.slots[seq];
+    const int lp = pos / p.page_size;
+    at_row = p.table[(long long)seq * p.table_stride + (lp % p.table_len)] * p.n_kv_heads * p.page_size + pos - lp * p.page_size;
+  }
+  __syncthreads();
+  if (!works) return;
   const T* src = reinterpret_cast<const T*>(p.proj) + ch0;
   const bool word = p.pairs_ok != 0;
   const int dkv = 2 * p.dim + p.vdim;
-  const int t_first = blockIdx.x * p.run, t_end = min(p.n_tokens, t_first + p.run);
-  // where the run's tokens lie: lane i looks up token i, so that the look-ups of a run wait for one another once
-  int at_r = 0, at_pos = 0, at_slot = 0, at_row = 0;
-  if (t_first + lane < t_end) {
-    const int t = t_first + lane, seq = p.token_seq[t];
-    at_pos = p.positions[t];
-    at_r = t - p.seq_start[seq];
-    at_slot = p.slots[seq];
-    const int lp = at_pos / p.page_size;
-    at_row = p.table[(long long)seq * p.table_stride + (lp % p.table_len)] * p.n_kv_heads * p.page_size + at_pos - lp * p.page_size;
-  }
+  float2 past[TAPS > 1 ? TAPS - 1 : 1][PJ];        // the inputs before the token, the newest last
   for (int t = t_first; t < t_end; ++t) {
-    const int r = __shfl_sync(0xffffffffu, at_r, t - t_first), pos = __shfl_sync(0xffffffffu, at_pos, t - t_first);
-    const int slot = __shfl_sync(0xffffffffu, at_slot, t - t_first);
+    const int r = __shfl_sync(0xffffffffu, at_r, t - t_first), slot = __shfl_sync(0xffffffffu, at_slot, t - t_first);
     const long long pool_row = __shfl_sync(0xffffffffu, at_row, t - t_first);
     float* kept = p.state + (long long)slot * (taps - 1) * channels + ch0;
     float2 y[PJ];
     float ss = 0.f;
+    // the input `back` tokens before the sequence's r-th of this step, at channel c
+    auto input = [&](int back, int c) {
+      const bool two = c + 1 < len;
+      if (back <= r) return da_pair<T>(src + (long long)(t - back) * p.row_stride + c, two, word);
+      const float* cell = kept + (long long)(taps - 1 + r - back) * channels + c;
+      return make_float2(cell[0], two ? cell[1] : 0.f);
+    };
 #pragma unroll
     for (int j = 0; j < PJ; ++j) {
       const int c = 2 * (lane + 32 * j);
-      const bool one = c < len, two = c + 1 < len;
-      float2 acc = make_float2(0.f, 0.f);
-      auto tap = [&](int k, float2 wk) {
-        const int back = taps - 1 - k;
-        float2 u = make_float2(0.f, 0.f);
-        if (one) {
-          if (back <= r) {
-            u = da_pair<T>(src + (long long)(t - back) * p.row_stride + c, two, word);
-          } else {
-            const float* cell = kept + (long long)(taps - 1 + r - back) * channels + c;
-            u = make_float2(cell[0], two ? cell[1] : 0.f);
-          }
-        }
-        acc.x = fmaf(wk.x, u.x, acc.x);
-        acc.y = fmaf(wk.y, u.y, acc.y);
-      };
+      const bool one = c < len;
+      float2 acc = make_float2(0.f, 0.f), u = make_float2(0.f, 0.f);
+      if (one) u = input(0, c);
       if (TAPS > 0) {
+        if (TAPS > 1 && (t == t_first || r == 0)) {
 #pragma unroll
-        for (int k = 0; k < (TAPS > 0 ? TAPS : 1); ++k) tap(k, w[k][j]);
-      } else {
+          for (int k = 0; k < TAPS - 1; ++k) past[k][j] = one ? input(TAPS - 1 - k, c) : make_float2(0.f, 0.f);
+        }
+#pragma unroll
+        for (int k = 0; k < TAPS - 1; ++k) {
+          acc.x = fmaf(w[k][j].x, past[k][j].x, acc.x);
+          acc.y = fmaf(w[k][j].y, past[k][j].y, acc.y);
+        }
+        acc.x = fmaf(w[TAPS > 0 ? TAPS - 1 : 0][j].x, u.x, acc.x);
+        acc.y = fmaf(w[TAPS > 0 ? TAPS - 1 : 0][j].y, u.y, acc.y);
+#pragma unroll
+        for (int k = 0; k + 1 < TAPS - 1; ++k) past[k][j] = past[k + 1][j];
+        if (TAPS > 1) past[TAPS > 1 ? TAPS - 2 : 0][j] = u;
+      } else if (one) {
         for (int k = 0; k < taps; ++k) {
           const float* wk = p.conv + (long long)k * channels + ch0 + c;
-          tap(k, one ? make_float2(wk[0], two ? wk[1] : 0.f) : make_float2(0.f, 0.f));
+          const float2 x = k == taps - 1 ? u : input(taps - 1 - k, c);
+          acc.x = fmaf(wk[0], x.x, acc.x);
+          acc.y = fmaf(c + 1 < len ? wk[1] : 0.f, x.y, acc.y);
         }
       }
       y[j] = acc;
       ss = fmaf(acc.x, acc.x, fmaf(acc.y, acc.y, ss));
-      if (p.shift_state && one) {
+      if (p.shift_state && one && taps > 1) {
         // one token a sequence: nobody else reads these channels of the sequence's state
         for (int k = 0; k + 1 < taps - 1; ++k) {
           kept[(long long)k * channels + c] = kept[(long long)(k + 1) * channels + c];
-          if (two) kept[(long long)k * channels + c + 1] = kept[(long long)(k + 1) * channels + c + 1];
+          if (c + 1 < len) kept[(long long)k * channels + c + 1] = kept[(long long)(k + 1) * channels + c + 1];
         }
-        if (taps > 1) {
-          const float2 u = da_pair<T>(src + (long long)t * p.row_stride + c, two, word);
-          kept[(long long)(taps - 2) * channels + c] = u.x;
-          if (two) kept[(long long)(taps - 2) * channels + c + 1] = u.y;
-        }
+        kept[(long long)(taps - 2) * channels + c] = u.x;
+        if (c + 1 < len) kept[(long long)(taps - 2) * channels + c + 1] = u.y;
       }
     }
     T* dst;
     if (is_q) {
       dst = reinterpret_cast<T*>(p.q_out) + (long long)t * q_units * p.q_pad + (long long)unit * p.q_pad;
     } else {
-      const int g = is_k ? (unit - q_units) >> 1 : unit - q_units - k_units;
+      const int g = is_k ? (unit - q_units) >> 1 : v_head;
       dst = reinterpret_cast<T*>(p.pool) + (pool_row + (long long)g * p.page_size) * dkv +
-            (is_k ? ((unit - q_units) & 1) * p.dim : 2 * p.dim);
+            (is_k ? ((unit - q_units) & 1) * p.dim : 2 * p.dim + v_first);
     }
     const float inv = weight != nullptr ? 1.f / sqrtf(warp_sum(ss) / (float)len + p.eps) : 1.f;
 #pragma unroll
@@ -163,17 +191,13 @@ __global__ void __launch_bounds__(128) differential_prep_kernel(DiffPrepArgs p) 
       const int c = 2 * (lane + 32 * j);
       if (c >= len) continue;
       float u = y[j].x * inv * gain[j].x, v = y[j].y * inv * gain[j].y;
-      if ((is_q || is_k) && c < p.rot_dims) {
-        float sn, cs;
-        sincosf((float)pos * freq[j], &sn, &cs);
-        sn *= p.rot_size;
-        cs *= p.rot_size;
-        const float a = u * cs - v * sn;
-        v = v * cs + u * sn;
+      if (!is_v && c < p.rot_dims) {
+        const float2 cs = turn[(t - t_first) * half + (c >> 1)];
+        const float a = u * cs.x - v * cs.y;
+        v = v * cs.x + u * cs.y;
         u = a;
       }
-      dst[c] = from_float<T>(u);
-      if (c + 1 < len) dst[c + 1] = from_float<T>(v);
+      da_store_pair(dst + c, u, v, c + 1 < len, word);
     }
     if (is_q)
       for (int c = len + lane; c < p.q_pad; c += 32) dst[c] = from_float<T>(0.f);
@@ -464,11 +488,17 @@ differential_combine_kernel(const float* __restrict__ parts, int n_splits, const
 
 template <typename T, int TAPS>
 static int launch_differential_prep(const DiffPrepArgs& p, cudaStream_t stream) {
-  const int units = 2 * p.n_heads + 3 * p.n_kv_heads, longest = p.dim > p.vdim ? p.dim : p.vdim;
-  const dim3 grid((p.n_tokens + p.run - 1) / p.run, (units + 3) / 4), block(128);
-  if (longest <= 64) BT_PDL_OK("differential_prep", launch_pdl(differential_prep_kernel<T, TAPS, 1>, grid, block, 0, stream, 1, p));
-  else if (longest <= 128) BT_PDL_OK("differential_prep", launch_pdl(differential_prep_kernel<T, TAPS, 2>, grid, block, 0, stream, 1, p));
-  else BT_PDL_OK("differential_prep", launch_pdl(differential_prep_kernel<T, TAPS, 4>, grid, block, 0, stream, 1, p));
+#define BT_DP(PJ)                                                                                                       \
+  do {                                                                                                                  \
+    const int units = 2 * (p.n_heads + p.n_kv_heads) + p.n_kv_heads * ((p.vdim + 64 * PJ - 1) / (64 * PJ));             \
+    const dim3 grid((p.n_tokens + p.run - 1) / p.run, (units + DA_PREP_WARPS - 1) / DA_PREP_WARPS);                     \
+    BT_PDL_OK("differential_prep", launch_pdl(differential_prep_kernel<T, TAPS, PJ>, grid, dim3(DA_PREP_WARPS * 32),    \
+                                              (size_t)p.run * (p.rot_dims / 2) * sizeof(float2), stream, 1, p));        \
+  } while (0)
+  if (p.dim <= 64) BT_DP(1);
+  else if (p.dim <= 128) BT_DP(2);
+  else BT_DP(4);
+#undef BT_DP
   return 0;
 }
 
@@ -577,10 +607,11 @@ extern "C" int bt_differential_prep(const void* proj, long long row_stride, cons
            n_kv_heads, dim, vdim, rot_dims, taps, DA_MAX_TAPS);
   if (n_tokens == 0) return 0;
   const int elem = dtype == kF32 ? 4 : 2;
-  const int words = row_stride % 2 == 0 && dim % 2 == 0 && vdim % 2 == 0 && (unsigned long long)proj % (2 * elem) == 0;
+  auto pairs = [&](const void* ptr) { return (unsigned long long)ptr % (2 * elem) == 0; };
+  const int words = row_stride % 2 == 0 && dim % 2 == 0 && vdim % 2 == 0 && q_pad % 2 == 0 && pairs(proj) && pairs(pool) && pairs(q_out);
   DiffPrepArgs p{proj, row_stride, conv, state, slots, seq_start, token_seq, positions, table, q_weight, k_weight, inv_freq, eps,
                  rot_size, rot_dims, taps, table_stride, table_len, page_size, pool, q_out, n_tokens, n_heads, n_kv_heads, dim,
-                 vdim, q_pad, n_tokens <= 256 ? 1 : 8, max_new == 1, words};
+                 vdim, q_pad, n_tokens <= 256 ? 1 : DA_RUN, max_new == 1, words};
   if (dtype == kF32) return run_differential_prep<float>(p, n_seqs, stream);
   if (dtype == kBF16) return run_differential_prep<__nv_bfloat16>(p, n_seqs, stream);
   return fail("differential_prep: unknown dtype %d", dtype);
