@@ -31,7 +31,6 @@ struct DiffPrepArgs {
   void* pool;                      // [pages][kv_heads][page_size][2 dim + vdim]
   void* q_out;                     // rows of 2 heads q_pad channels
   int n_tokens, n_heads, n_kv_heads, dim, vdim, q_pad;
-  int run;                         // consecutive tokens a warp takes
   int shift_state;                 // every sequence brings one token: the kernel moves the state on itself
   int pairs_ok;                    // two adjacent channels may be read and written as one word
 };
@@ -61,15 +60,14 @@ __device__ __forceinline__ void da_store_pair(__nv_bfloat16* p, float a, float b
 }
 
 constexpr int DA_PREP_WARPS = 8;
-constexpr int DA_RUN = 8;          // consecutive tokens a warp takes at most
 
-// A warp takes one unit (a map of a query or key head, or 64 PJ channels of a value head) of `run` consecutive tokens; a lane
-// owns PJ channel pairs of it, 64 channels apart.  Where TAPS says how many taps there are (0: any number), taps and the
-// last TAPS - 1 inputs stay in registers, so every input is read once a run.  The block's warps take the same tokens: sines
-// and cosines of the run are formed once for all of them.
-template <typename T, int TAPS, int PJ>
+// A warp takes one unit (a map of a query or key head, or 64 PJ channels of a value head) of RUN consecutive tokens; a lane
+// owns PJ channel pairs of it, 64 channels apart.  The run's inputs are asked for together; where TAPS says how many taps
+// there are (0: any number), taps and the inputs before the run stay in registers too, so every input is read once a run.
+// The block's warps take the same tokens: sines and cosines of the run are formed once for all of them.
+template <typename T, int TAPS, int PJ, int RUN>
 __global__ void __launch_bounds__(DA_PREP_WARPS * 32) differential_prep_kernel(DiffPrepArgs p) {
-  extern __shared__ float2 turn[];       // [run][rot_dims / 2]: (cosine, sine) times rot_size
+  extern __shared__ float2 turn[];       // [RUN][rot_dims / 2]: (cosine, sine) times rot_size
   const int lane = threadIdx.x & 31;
   const int v_pieces = (p.vdim + 64 * PJ - 1) / (64 * PJ);
   const int q_units = 2 * p.n_heads, k_units = 2 * p.n_kv_heads, units = q_units + k_units + p.n_kv_heads * v_pieces;
@@ -101,7 +99,7 @@ __global__ void __launch_bounds__(DA_PREP_WARPS * 32) differential_prep_kernel(D
     }
   }
   pdl_wait();
-  const int t_first = blockIdx.x * p.run, t_end = min(p.n_tokens, t_first + p.run), half = p.rot_dims >> 1;
+  const int t_first = blockIdx.x * RUN, t_end = min(p.n_tokens, t_first + RUN), half = p.rot_dims >> 1;
   for (int i = threadIdx.x; i < (t_end - t_first) * half; i += DA_PREP_WARPS * 32) {
     const int t = i / half, pair = i - t * half;
     float sn, cs;
@@ -110,7 +108,7 @@ __global__ void __launch_bounds__(DA_PREP_WARPS * 32) differential_prep_kernel(D
   }
   // where the run's tokens lie: lane i looks up token i, so that the look-ups of a run wait for one another once
   int at_r = 0, at_slot = 0, at_row = 0;
-  if (t_first + lane < t_end) {
+  if (lane < t_end - t_first) {
     const int t = t_first + lane, seq = p.token_seq[t], pos = p.positions[t];
     at_r = t - p.seq_start[seq];
     at_slot = p.slots[seq];
@@ -123,9 +121,21 @@ __global__ void __launch_bounds__(DA_PREP_WARPS * 32) differential_prep_kernel(D
   const bool word = p.pairs_ok != 0;
   const int dkv = 2 * p.dim + p.vdim;
   float2 past[TAPS > 1 ? TAPS - 1 : 1][PJ];        // the inputs before the token, the newest last
-  for (int t = t_first; t < t_end; ++t) {
-    const int r = __shfl_sync(0xffffffffu, at_r, t - t_first), slot = __shfl_sync(0xffffffffu, at_slot, t - t_first);
-    const long long pool_row = __shfl_sync(0xffffffffu, at_row, t - t_first);
+  float2 own[RUN][PJ];                             // the run's inputs
+#pragma unroll
+  for (int i = 0; i < RUN; ++i)
+#pragma unroll
+    for (int j = 0; j < PJ; ++j) {
+      const int c = 2 * (lane + 32 * j);
+      own[i][j] = t_first + i < t_end && c < len ? da_pair<T>(src + (long long)(t_first + i) * p.row_stride + c, c + 1 < len, word)
+                                                 : make_float2(0.f, 0.f);
+    }
+#pragma unroll
+  for (int i = 0; i < RUN; ++i) {
+    const int t = t_first + i;
+    if (t >= t_end) break;
+    const int r = __shfl_sync(0xffffffffu, at_r, i), slot = __shfl_sync(0xffffffffu, at_slot, i);
+    const long long pool_row = __shfl_sync(0xffffffffu, at_row, i);
     float* kept = p.state + (long long)slot * (taps - 1) * channels + ch0;
     float2 y[PJ];
     float ss = 0.f;
@@ -140,10 +150,10 @@ __global__ void __launch_bounds__(DA_PREP_WARPS * 32) differential_prep_kernel(D
     for (int j = 0; j < PJ; ++j) {
       const int c = 2 * (lane + 32 * j);
       const bool one = c < len;
-      float2 acc = make_float2(0.f, 0.f), u = make_float2(0.f, 0.f);
-      if (one) u = input(0, c);
+      float2 acc = make_float2(0.f, 0.f);
+      const float2 u = own[i][j];
       if (TAPS > 0) {
-        if (TAPS > 1 && (t == t_first || r == 0)) {
+        if (TAPS > 1 && (i == 0 || r == 0)) {
 #pragma unroll
           for (int k = 0; k < TAPS - 1; ++k) past[k][j] = one ? input(TAPS - 1 - k, c) : make_float2(0.f, 0.f);
         }
@@ -192,7 +202,7 @@ __global__ void __launch_bounds__(DA_PREP_WARPS * 32) differential_prep_kernel(D
       if (c >= len) continue;
       float u = y[j].x * inv * gain[j].x, v = y[j].y * inv * gain[j].y;
       if (!is_v && c < p.rot_dims) {
-        const float2 cs = turn[(t - t_first) * half + (c >> 1)];
+        const float2 cs = turn[i * half + (c >> 1)];
         const float a = u * cs.x - v * cs.y;
         v = v * cs.x + u * cs.y;
         u = a;
@@ -225,19 +235,24 @@ differential_state_kernel(const T* __restrict__ proj, long long row_stride, floa
   }
 }
 
-// A number of the cache's element type read from shared memory as a 4-byte piece.
-template <typename T> struct DaPiece;
-template <> struct DaPiece<float> {
-  static constexpr int N = 1;
-  __device__ static void read(const float* p, float (&o)[2]) { o[0] = *p; o[1] = 0.f; }
-};
-template <> struct DaPiece<__nv_bfloat16> {
-  static constexpr int N = 2;
-  __device__ static void read(const __nv_bfloat16* p, float (&o)[2]) {
-    const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
-    o[0] = f.x; o[1] = f.y;
+// 16 bytes of shared memory as numbers.
+__device__ __forceinline__ void da_piece(const float* p, float (&o)[4]) {
+  const float4 f = *reinterpret_cast<const float4*>(p);
+  o[0] = f.x; o[1] = f.y; o[2] = f.z; o[3] = f.w;
+}
+__device__ __forceinline__ void da_piece(const __nv_bfloat16* p, float (&o)[8]) {
+  const uint4 raw = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 f = __bfloat1622float2(h[i]);
+    o[2 * i] = f.x;
+    o[2 * i + 1] = f.y;
   }
-};
+}
+__device__ __forceinline__ void da_copy16(void* smem, const void* gmem) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((unsigned)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
 
 struct TwoMapArgs {
   const void* q;                    // rows of 2 heads dim_pad channels
@@ -259,12 +274,11 @@ struct TwoMapArgs {
 template <typename T, int ROWS, int DVL>
 __global__ void __launch_bounds__(256) two_map_attention_kernel(TwoMapArgs p) {
   extern __shared__ __align__(16) float smem[];
-  constexpr int PN = DaPiece<T>::N;
   const int n_warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int dim = p.dim, vdim = p.vdim, ks = p.ks, dkv = 2 * dim + vdim;
   float* q_s = smem;                                                                // [dim][ROWS]
-  const int tile_words = (DA_TK * (ks + vdim) * (int)sizeof(T) + 3) / 4;
-  T* k_s = reinterpret_cast<T*>(q_s + ROWS * dim + (size_t)warp * tile_words);      // this warp's [DA_TK][ks]: both keys
+  const int tile_words = (DA_TK * (ks + vdim) * (int)sizeof(T) + 15) / 16 * 4;
+  T* k_s = reinterpret_cast<T*>(q_s + (ROWS * dim + 3) / 4 * 4 + (size_t)warp * tile_words);   // this warp's [DA_TK][ks]: both keys
   T* v_s = k_s + DA_TK * ks;                                                        // this warp's [DA_TK][vdim]
   pdl_trigger();
   pdl_wait();
@@ -275,12 +289,6 @@ __global__ void __launch_bounds__(256) two_map_attention_kernel(TwoMapArgs p) {
   const int h0 = g * group_heads + head_tile * (ROWS / 2);
   const int rows = 2 * min(ROWS / 2, (g + 1) * group_heads - h0);
   const int seq = p.token_seq[token], pos = p.positions[token];
-  const T* q = reinterpret_cast<const T*>(p.q) + token * p.q_row_stride + (long long)2 * h0 * p.q_pad;
-  for (int i = threadIdx.x; i < ROWS * dim; i += blockDim.x) {
-    const int r = i / dim, d = i - r * dim;
-    q_s[d * ROWS + r] = r < rows ? to_float(q[(long long)r * p.q_pad + d]) : 0.f;
-  }
-  __syncthreads();
   float acc[ROWS][DVL], top[ROWS], sum[ROWS];
 #pragma unroll
   for (int r = 0; r < ROWS; ++r) {
@@ -292,23 +300,18 @@ __global__ void __launch_bounds__(256) two_map_attention_kernel(TwoMapArgs p) {
   const int n_tiles = pos / DA_TK + 1, per_split = (n_tiles + p.n_splits - 1) / p.n_splits;
   const int tile_end = min(n_tiles, (split + 1) * per_split);
   constexpr int V = 16 / (int)sizeof(T);
-  const bool pieces_ok = dim % V == 0 && vdim % V == 0 && ks % PN == 0 && (reinterpret_cast<unsigned long long>(p.pool) & 15) == 0;
-  for (int tile = split * per_split + warp; tile < tile_end; tile += n_warps) {
-    const int j0 = tile * DA_TK;
-    __syncwarp();          // the lanes are done with the tile before
-    // (a tile never straddles a page, and a key head's rows lie one after another in it.  Positions past the token's own
-    // hold finite numbers of whoever had the page before: their weights are zero)
-    const int lp = j0 / p.page_size;
+  const bool pieces_ok = dim % V == 0 && vdim % V == 0 && (reinterpret_cast<unsigned long long>(p.pool) & 15) == 0;
+  // (a tile never straddles a page, and a key head's rows lie one after another in it.  Positions past the token's own hold
+  // finite numbers of whoever had the page before: their weights are zero)
+  auto fetch = [&](int tile) {
+    const int j0 = tile * DA_TK, lp = j0 / p.page_size;
     const long long page = p.table[(long long)seq * p.table_stride + (lp % p.table_len)];
     const T* src = reinterpret_cast<const T*>(p.pool) + ((page * p.n_kv_heads + g) * p.page_size + (j0 - lp * p.page_size)) * dkv;
     if (pieces_ok) {
       const int per_row = dkv / V, n_pieces = DA_TK * per_row;
-#pragma unroll 8
       for (int i = lane; i < n_pieces; i += 32) {
         const int kk = i / per_row, d0 = (i - kk * per_row) * V;
-        const uint4 raw = *reinterpret_cast<const uint4*>(src + (long long)i * V);
-        uint32_t* dst = reinterpret_cast<uint32_t*>(d0 < 2 * dim ? k_s + kk * ks + d0 : v_s + kk * vdim + (d0 - 2 * dim));
-        dst[0] = raw.x; dst[1] = raw.y; dst[2] = raw.z; dst[3] = raw.w;
+        da_copy16(d0 < 2 * dim ? k_s + kk * ks + d0 : v_s + kk * vdim + (d0 - 2 * dim), src + (long long)i * V);
       }
     } else {
       for (int i = lane; i < DA_TK * dkv; i += 32) {
@@ -316,6 +319,22 @@ __global__ void __launch_bounds__(256) two_map_attention_kernel(TwoMapArgs p) {
         if (d < 2 * dim) k_s[kk * ks + d] = src[i]; else v_s[kk * vdim + d - 2 * dim] = src[i];
       }
     }
+  };
+  const int tile_first = split * per_split + warp;
+  if (tile_first < tile_end) fetch(tile_first);          // (the queries are laid out while the first tile is on its way)
+  const T* q = reinterpret_cast<const T*>(p.q) + token * p.q_row_stride + (long long)2 * h0 * p.q_pad;
+  for (int i = threadIdx.x; i < ROWS * dim; i += blockDim.x) {
+    const int r = i / dim, d = i - r * dim;
+    q_s[d * ROWS + r] = r < rows ? to_float(q[(long long)r * p.q_pad + d]) : 0.f;
+  }
+  __syncthreads();
+  for (int tile = tile_first; tile < tile_end; tile += n_warps) {
+    const int j0 = tile * DA_TK;
+    if (tile != tile_first) {
+      __syncwarp();          // the lanes are done with the tile before
+      fetch(tile);
+    }
+    asm volatile("cp.async.wait_all;\n" ::: "memory");
     __syncwarp();
     float s[ROWS];
 #pragma unroll
@@ -341,14 +360,14 @@ __global__ void __launch_bounds__(256) two_map_attention_kernel(TwoMapArgs p) {
       }
     };
     int d = 0;
-    if (ks % PN == 0 && dim % PN == 0) {
-#pragma unroll 4
-      for (; d + PN <= dim; d += PN) {
-        float k1[2], k2[2];
-        DaPiece<T>::read(krow + d, k1);
-        DaPiece<T>::read(krow + dim + d, k2);
+    if (pieces_ok) {
+#pragma unroll 2
+      for (; d < dim; d += V) {
+        float k1[V], k2[V];
+        da_piece(krow + d, k1);
+        da_piece(krow + dim + d, k2);
 #pragma unroll
-        for (int u = 0; u < PN; ++u) take(d + u, k1[u], k2[u]);
+        for (int u = 0; u < V; ++u) take(d + u, k1[u], k2[u]);
       }
     }
     for (; d < dim; ++d) take(d, to_float(krow[d]), to_float(krow[dim + d]));
@@ -380,7 +399,7 @@ __global__ void __launch_bounds__(256) two_map_attention_kernel(TwoMapArgs p) {
   }
   // the warps' results, joined in warp order (the tiles' shared memory is free now)
   __syncthreads();
-  float* sums = q_s + ROWS * dim;                              // [n_warps][ROWS][vdim + 2]
+  float* sums = q_s + (ROWS * dim + 3) / 4 * 4;                // [n_warps][ROWS][vdim + 2]
 #pragma unroll
   for (int r = 0; r < ROWS; ++r) {
     float* cell = sums + ((size_t)warp * ROWS + r) * (vdim + 2);
@@ -431,45 +450,59 @@ differential_combine_kernel(const float* __restrict__ parts, int n_splits, const
   const long long token = item / n_heads;
   const int head = (int)(item - token * n_heads);
   float o[2][DVL];
+  const long long row = token * 2 * n_heads + 2 * head;          // the second map's row follows
+  if (n_splits == 1) {
 #pragma unroll
-  for (int m = 0; m < 2; ++m) {
-    const long long row = token * 2 * n_heads + 2 * head + m;
-    if (n_splits == 1) {
+    for (int m = 0; m < 2; ++m)
 #pragma unroll
       for (int j = 0; j < DVL; ++j) {
         const int c = lane + 32 * j;
-        o[m][j] = c < vdim ? parts[row * vdim + c] : 0.f;
+        o[m][j] = c < vdim ? parts[(row + m) * vdim + c] : 0.f;
       }
-      continue;
-    }
-    const float* src = parts + row * n_splits * (vdim + 2);
-    float w[DA_MAX_SPLITS / 32], high = -INFINITY, denom = 0.f;
+  } else {
+    const int step = vdim + 2;
+    const float* src = parts + row * n_splits * step;
+    const long long second = (long long)n_splits * step;
+    float w[2][DA_MAX_SPLITS / 32], l[2][DA_MAX_SPLITS / 32], denom[2] = {0.f, 0.f};
 #pragma unroll
-    for (int i = 0; i < DA_MAX_SPLITS / 32; ++i) {
-      const int s = lane + 32 * i;
-      w[i] = s < n_splits ? src[(long long)s * (vdim + 2) + vdim] : -INFINITY;
-      high = fmaxf(high, w[i]);
-    }
-    high = warp_max(high);
+    for (int m = 0; m < 2; ++m)
 #pragma unroll
-    for (int i = 0; i < DA_MAX_SPLITS / 32; ++i) {
-      const int s = lane + 32 * i;
-      w[i] = w[i] == -INFINITY ? 0.f : expf(w[i] - high);
-      if (s < n_splits) denom = fmaf(w[i], src[(long long)s * (vdim + 2) + vdim + 1], denom);
-    }
-    denom = warp_sum(denom);
+      for (int i = 0; i < DA_MAX_SPLITS / 32; ++i) {
+        const int s = lane + 32 * i;
+        w[m][i] = s < n_splits ? src[m * second + (long long)s * step + vdim] : -INFINITY;
+        l[m][i] = s < n_splits ? src[m * second + (long long)s * step + vdim + 1] : 0.f;
+      }
 #pragma unroll
-    for (int j = 0; j < DVL; ++j) o[m][j] = 0.f;
+    for (int m = 0; m < 2; ++m) {
+      float high = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < DA_MAX_SPLITS / 32; ++i) high = fmaxf(high, w[m][i]);
+      high = warp_max(high);
+#pragma unroll
+      for (int i = 0; i < DA_MAX_SPLITS / 32; ++i) {
+        w[m][i] = w[m][i] == -INFINITY ? 0.f : expf(w[m][i] - high);
+        denom[m] = fmaf(w[m][i], l[m][i], denom[m]);
+      }
+      denom[m] = warp_sum(denom[m]);
+#pragma unroll
+      for (int j = 0; j < DVL; ++j) o[m][j] = 0.f;
+    }
+#pragma unroll 4
     for (int s = 0; s < n_splits; ++s) {
-      const float f = __shfl_sync(0xffffffffu, s < 32 ? w[0] : w[DA_MAX_SPLITS / 32 - 1], s & 31);
 #pragma unroll
-      for (int j = 0; j < DVL; ++j) {
-        const int c = lane + 32 * j;
-        if (c < vdim) o[m][j] = fmaf(f, src[(long long)s * (vdim + 2) + c], o[m][j]);
+      for (int m = 0; m < 2; ++m) {
+        const float f = __shfl_sync(0xffffffffu, s < 32 ? w[m][0] : w[m][DA_MAX_SPLITS / 32 - 1], s & 31);
+#pragma unroll
+        for (int j = 0; j < DVL; ++j) {
+          const int c = lane + 32 * j;
+          if (c < vdim) o[m][j] = fmaf(f, src[m * second + (long long)s * step + c], o[m][j]);
+        }
       }
     }
 #pragma unroll
-    for (int j = 0; j < DVL; ++j) o[m][j] /= denom;
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int j = 0; j < DVL; ++j) o[m][j] /= denom[m];
   }
   const float lambda = share[0];
   float ss = 0.f;
@@ -486,19 +519,26 @@ differential_combine_kernel(const float* __restrict__ parts, int n_splits, const
   }
 }
 
+// (a warp takes one token in steps of few tokens, else as many as its registers hold the inputs of)
 template <typename T, int TAPS>
 static int launch_differential_prep(const DiffPrepArgs& p, cudaStream_t stream) {
-#define BT_DP(PJ)                                                                                                       \
+#define BT_DP_RUN(PJ, RUN)                                                                                              \
   do {                                                                                                                  \
     const int units = 2 * (p.n_heads + p.n_kv_heads) + p.n_kv_heads * ((p.vdim + 64 * PJ - 1) / (64 * PJ));             \
-    const dim3 grid((p.n_tokens + p.run - 1) / p.run, (units + DA_PREP_WARPS - 1) / DA_PREP_WARPS);                     \
-    BT_PDL_OK("differential_prep", launch_pdl(differential_prep_kernel<T, TAPS, PJ>, grid, dim3(DA_PREP_WARPS * 32),    \
-                                              (size_t)p.run * (p.rot_dims / 2) * sizeof(float2), stream, 1, p));        \
+    const dim3 grid((p.n_tokens + RUN - 1) / RUN, (units + DA_PREP_WARPS - 1) / DA_PREP_WARPS);                         \
+    auto kernel = differential_prep_kernel<T, TAPS, PJ, RUN>;                                                           \
+    BT_PDL_OK("differential_prep", launch_pdl(kernel, grid, dim3(DA_PREP_WARPS * 32),                                   \
+                                              (size_t)RUN * (p.rot_dims / 2) * sizeof(float2), stream, 1, p));          \
   } while (0)
-  if (p.dim <= 64) BT_DP(1);
-  else if (p.dim <= 128) BT_DP(2);
-  else BT_DP(4);
+#define BT_DP(PJ, RUN)                                                                                                  \
+  do {                                                                                                                  \
+    if (p.n_tokens <= 256) BT_DP_RUN(PJ, 1); else BT_DP_RUN(PJ, RUN);                                                   \
+  } while (0)
+  if (p.dim <= 64) BT_DP(1, 8);
+  else if (p.dim <= 128) BT_DP(2, 4);
+  else BT_DP(4, 2);
 #undef BT_DP
+#undef BT_DP_RUN
   return 0;
 }
 
@@ -506,8 +546,6 @@ template <typename T>
 static int run_differential_prep(const DiffPrepArgs& p, int n_seqs, cudaStream_t stream) {
   int rc;
   switch (p.taps) {
-    case 1: rc = launch_differential_prep<T, 1>(p, stream); break;
-    case 2: rc = launch_differential_prep<T, 2>(p, stream); break;
     case 3: rc = launch_differential_prep<T, 3>(p, stream); break;
     case 4: rc = launch_differential_prep<T, 4>(p, stream); break;
     default: rc = launch_differential_prep<T, 0>(p, stream);
@@ -527,15 +565,15 @@ static TwoMapShape two_map_shape(int group_heads, int dim, int vdim, int elem) {
   TwoMapShape s;
   s.rows = group_heads <= 1 ? 2 : (group_heads <= 2 ? 4 : 8);
   s.head_tiles = (group_heads + s.rows / 2 - 1) / (s.rows / 2);
-  // a key row's length in shared memory: whole 4-byte pieces, an odd number of them, so that the lanes' rows start in
-  // different banks
-  const int per_word = 4 / elem;
-  s.ks = (2 * dim + per_word - 1) / per_word * per_word;
-  if ((s.ks / per_word) % 2 == 0) s.ks += per_word;
-  const size_t tile_words = ((size_t)DA_TK * (s.ks + vdim) * elem + 3) / 4;
+  // a key row's length in shared memory: whole 16-byte pieces, an odd number of them, so that the eight lanes of a 16-byte
+  // read meet every bank once
+  const int piece = 16 / elem;
+  s.ks = (2 * dim + piece - 1) / piece * piece;
+  if ((s.ks / piece) % 2 == 0) s.ks += piece;
+  const size_t tile_words = ((size_t)DA_TK * (s.ks + vdim) * elem + 15) / 16 * 4;
   auto bytes = [&](int w) {
     const size_t tiles = (size_t)w * tile_words, sums = (size_t)w * s.rows * (vdim + 2);
-    return ((size_t)s.rows * dim + (tiles > sums ? tiles : sums)) * sizeof(float);
+    return (((size_t)s.rows * dim + 3) / 4 * 4 + (tiles > sums ? tiles : sums)) * sizeof(float);
   };
   s.warps = 4;
   while (s.warps > 1 && bytes(s.warps) > 160 * 1024) s.warps >>= 1;
@@ -611,7 +649,7 @@ extern "C" int bt_differential_prep(const void* proj, long long row_stride, cons
   const int words = row_stride % 2 == 0 && dim % 2 == 0 && vdim % 2 == 0 && q_pad % 2 == 0 && pairs(proj) && pairs(pool) && pairs(q_out);
   DiffPrepArgs p{proj, row_stride, conv, state, slots, seq_start, token_seq, positions, table, q_weight, k_weight, inv_freq, eps,
                  rot_size, rot_dims, taps, table_stride, table_len, page_size, pool, q_out, n_tokens, n_heads, n_kv_heads, dim,
-                 vdim, q_pad, n_tokens <= 256 ? 1 : DA_RUN, max_new == 1, words};
+                 vdim, q_pad, max_new == 1, words};
   if (dtype == kF32) return run_differential_prep<float>(p, n_seqs, stream);
   if (dtype == kBF16) return run_differential_prep<__nv_bfloat16>(p, n_seqs, stream);
   return fail("differential_prep: unknown dtype %d", dtype);
