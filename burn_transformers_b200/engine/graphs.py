@@ -185,6 +185,9 @@ class DecodeGraph:
         # a recording must find every piece of scratch at a fixed address: size the workspace for a whole step
         # before recording, and let it grow no more
         first = self._settle(first)
+        # (a part met before one that has no phase launches its kernels for real: they write into the scratch memory that
+        # this step's result lies in)
+        first = first.clone()
         self.program = self._record_program()
         if self.program is not None and self.ws._retired:
             # the fused step needed more scratch than the separate kernels: make room, then record for good
